@@ -125,7 +125,7 @@ __device__ __forceinline__ float act_df(int kind, float x) {
 template <bool BF16, int KIND, bool LIMIT>
 __global__ void __launch_bounds__(256) glu_fwd_kernel(const uint16_t* __restrict__ x, uint16_t* __restrict__ y,
                                                       long long M, int F, int kind_arg, int gate_is_act,
-                                                      const int* __restrict__ row_limit) {
+                                                      const int* __restrict__ row_limit, long long ldx) {
   const int kind = KIND >= 0 ? KIND : kind_arg;
   const int vecs = F >> 3;
   const long long total = M * vecs;
@@ -141,8 +141,8 @@ __global__ void __launch_bounds__(256) glu_fwd_kernel(const uint16_t* __restrict
   // dead rows are not read: their loads go to row 0 instead (always inside the buffer), unconditionally, so that
   // the four loads are issued back to back; the select below discards what they return
   const bool live0 = !LIMIT || m0 < live, live1 = two && (!LIMIT || m1 < live);
-  const uint16_t* r0 = x + (size_t)(live0 ? m0 : 0) * 2 * F + v0 * 8;
-  const uint16_t* r1 = x + (size_t)(live1 ? m1 : 0) * 2 * F + v1 * 8;
+  const uint16_t* r0 = x + (live0 ? m0 : 0) * ldx + v0 * 8;
+  const uint16_t* r1 = x + (live1 ? m1 : 0) * ldx + v1 * 8;
   float f0[8], g0[8], f1[8], g1[8], o[8];
   ld8<BF16>(r0, f0);
   ld8<BF16>(r0 + F, g0);
@@ -579,17 +579,20 @@ ICB_API int icb_rope(const void* x, void* out, const int* pos_ids, int T, int nh
   return check_launch("rope");
 }
 
-// row_limit (optional, device int32): rows from *row_limit on are not read and get zeros.
+// row_limit (optional, device int32): rows from *row_limit on are not read and get zeros. ldx: pitch of x's rows
+// (0: 2 F, packed), a multiple of 8.
 ICB_API int icb_glu_fwd(const void* x, void* y, long long M, int F, int kind, int gate_is_act, int dtype,
-                        void* stream, const int* row_limit) {
+                        void* stream, const int* row_limit, long long ldx) {
   if (M <= 0) return 0;
-  if (F % 8) return -2;
+  if (ldx == 0) ldx = 2LL * F;
+  if (F % 8 || ldx % 8 || ldx < 2LL * F) return -2;
   const long long n = (M * (F / 8) + 1) / 2;
   const int th = 256;
   const int bl = (int)((n + th - 1) / th);
   const bool silu = kind == 3 && !gate_is_act;
+  const bool gelu = kind == 2 && !gate_is_act;
 #define ICB_GLU_FWD(B16, K, L) \
-  glu_fwd_kernel<B16, K, L><<<bl, th, 0, ICB_ST(stream)>>>(ICB_U16(x), ICB_U16M(y), M, F, kind, gate_is_act, row_limit)
+  glu_fwd_kernel<B16, K, L><<<bl, th, 0, ICB_ST(stream)>>>(ICB_U16(x), ICB_U16M(y), M, F, kind, gate_is_act, row_limit, ldx)
 #define ICB_GLU_FWD_L(B16, K)            \
   do {                                   \
     if (row_limit != nullptr) ICB_GLU_FWD(B16, K, true); \
@@ -597,6 +600,7 @@ ICB_API int icb_glu_fwd(const void* x, void* y, long long M, int F, int kind, in
   } while (0)
   if (dtype == kBF16) {
     if (silu) ICB_GLU_FWD_L(true, 3);
+    else if (gelu) ICB_GLU_FWD_L(true, 2);
     else ICB_GLU_FWD_L(true, -1);
   } else {
     if (silu) ICB_GLU_FWD_L(false, 3);

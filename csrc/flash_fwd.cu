@@ -1,5 +1,5 @@
 // Flash attention forward for sm_100a: causal / full, GQA, optional document
-// boundaries (cu_seqlens), head_dim 64 or 128, bf16 or fp16.
+// boundaries (cu_seqlens), sliding window, per-head output gate, head_dim 64 or 128, bf16 or fp16.
 //
 // One CTA owns 128 query rows of one head. Warp 0 streams K and V tiles (128 rows)
 // with TMA into 2-stage rings, warp 1 issues tcgen05.mma for S = Q K^T (TMEM,
@@ -36,6 +36,8 @@ struct FlashFwdArgs {
   const unsigned long long* drop_seed;  // device word; read when drop_thr > 0
   int drop_thr;                       // keep a probability when its hash byte >= drop_thr (0: no dropout)
   float drop_scale;                   // 256 / (256 - drop_thr)
+  int window;                         // causal only: query i sees keys j with i - j < window (0: no limit)
+  const float* gate;                  // [T, hq] factor of a head's output row, or null
 };
 
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -114,7 +116,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   if (qt >= num_q_tiles) return;
   const int q0 = qt * 128;
   const int n_kv_total = (seq_len + BN - 1) / BN;
-  const int n_kv = args.causal ? min((q0 + 128 + BN - 1) / BN, n_kv_total) : n_kv_total;
+  const int kv_end = args.causal ? min((q0 + 128 + BN - 1) / BN, n_kv_total) : n_kv_total;
+  // key tiles that end before the window of the tile's first query row are not visited
+  const int kv_first = args.window > 0 ? max(0, q0 - args.window + 1) / BN : 0;
+  const int n_kv = kv_end - kv_first;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -152,7 +157,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       for (int j = 0; j < n_kv; ++j) {
         const int s = j & 1;
         const uint32_t ph = (j >> 1) & 1;
-        const int t0 = seq_start + j * BN;
+        const int t0 = seq_start + (kv_first + j) * BN;
         mbar_wait(&k_empty[s], ph ^ 1, abort_flag, args.status, kTimeoutSmemEmpty);
         mbar_expect_tx(&k_full[s], L::kv_bytes);
 #pragma unroll
@@ -240,8 +245,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(&s_empty[s]);
-      const int kv0 = j * BN;
-      const bool need_mask = (args.causal && kv0 + BN > q0) || (kv0 + BN > seq_len);
+      const int kv0 = (kv_first + j) * BN;
+      const int kv_lo = args.window > 0 ? q_idx - args.window : -1;      // last key that this row no longer sees
+      const bool need_mask = (args.causal && kv0 + BN > q0) || (kv0 + BN > seq_len) ||
+                             (args.window > 0 && kv0 <= q0 + 127 - args.window);
       float m_tile = -INFINITY;
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
@@ -250,14 +257,14 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           float x = __uint_as_float(r[c][i]) * args.scale_log2;
           if (need_mask) {
             const int kv_idx = kv0 + c * 32 + i;
-            if (kv_idx >= seq_len || (args.causal && kv_idx > q_idx)) x = -INFINITY;
+            if (kv_idx >= seq_len || (args.causal && kv_idx > q_idx) || kv_idx <= kv_lo) x = -INFINITY;
           }
           r[c][i] = __float_as_uint(x);
           m_tile = fmaxf(m_tile, x);
         }
       }
-      float m_new = fmaxf(m_ref, m_tile);
-      if (m_new == -INFINITY) m_new = 0.f;
+      // -inf as long as a row has seen no visible key (its window may start in a later tile)
+      const float m_new = fmaxf(m_ref, m_tile);
       const bool grow = m_new > m_ref + 8.0f;
       const unsigned any_grow = __ballot_sync(0xffffffffu, grow);
       if (any_grow) {
@@ -289,6 +296,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const uint32_t php = (j / PS) & 1;
       if (j >= PS) mbar_wait(&p_empty[sp], php ^ 1, abort_flag, args.status, kTimeoutLocalFlag);
       uint8_t* prow = sP + sp * L::p_bytes + row * 128;
+      const float m_sub = m_ref == -INFINITY ? 0.f : m_ref;
       float lsum_tile = 0.f;
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
@@ -297,7 +305,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           float p[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            p[i] = fast_exp2(__uint_as_float(r[c][g * 8 + i]) - m_ref);
+            p[i] = fast_exp2(__uint_as_float(r[c][g * 8 + i]) - m_sub);
             lsum_tile += p[i];
           }
           if (dropout) {
@@ -330,9 +338,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const int last = n_kv - 1;
       mbar_wait(&p_empty[last % PS], (last / PS) & 1, abort_flag, args.status, kTimeoutTmemFull);
       tc_fence_after();
-      const float inv_l = l_sum > 0.f ? 1.0f / l_sum : 0.f;
       const bool valid = q_idx < seq_len;
       const long long tok = (long long)seq_start + q_idx;
+      float inv_l = l_sum > 0.f ? 1.0f / l_sum : 0.f;
+      if (args.gate != nullptr && valid) inv_l *= args.gate[(size_t)tok * args.hq + head];
       uint8_t* orow = reinterpret_cast<uint8_t*>(args.out) + ((size_t)tok * args.hq + head) * HD * 2;
 #pragma unroll
       for (int c = 0; c < HD / 32; ++c) {
@@ -414,12 +423,16 @@ using namespace icb;
 // [batch + 1]) gives document boundaries in the flat token stream; seq_len is then the maximum length.
 // dropout_p > 0 drops attention probabilities with probability round(256 p) / 256 under the mask that the
 // device word *dropout_seed selects (the backward pass must be given the same word).
+// window > 0 (causal only): a query's keys are the `window` tokens that end with itself. gate (optional, fp32 [T, hq]) multiplies a
+// head's output row.
 ICB_API int icb_flash_fwd(const void* q, const void* k, const void* v, void* out, float* lse, int batch, int seq_len,
                           long long total_tokens, int hq, int hkv, int hd, long long q_stride, long long kv_stride,
                           const int* cu_seqlens, int causal, float scale, int dtype, int* status, void* stream_,
-                          float dropout_p, const unsigned long long* dropout_seed, int wide) {
+                          float dropout_p, const unsigned long long* dropout_seed, int wide, int window,
+                          const float* gate) {
   if (hd != 64 && hd != 128) return -2;
   if (hq % hkv != 0) return -3;
+  if (window > 0 && !causal) return -5;
   if (batch <= 0 || seq_len <= 0) return 0;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   CUtensorMap tmQ, tmK, tmV;
@@ -442,6 +455,8 @@ ICB_API int icb_flash_fwd(const void* q, const void* k, const void* v, void* out
   if (a.drop_thr > 0 && dropout_seed == nullptr) return -4;
   a.drop_seed = dropout_seed;
   a.drop_scale = 256.0f / (256 - a.drop_thr);
+  a.window = window > 0 ? window : 0;
+  a.gate = gate;
   dim3 grid((seq_len + 127) / 128, hq, batch);
   if (bn == 64) {
     if (hd == 64) return launch_flash_fwd<64, 64>(tmQ, tmK, tmV, a, grid, stream);

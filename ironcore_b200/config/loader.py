@@ -53,7 +53,7 @@ def _merge_single_key_lists(node: Any) -> Any:
     if isinstance(node, dict):
         return {k: _merge_single_key_lists(v) for k, v in node.items()}
     if isinstance(node, list):
-        if node and all(isinstance(it, dict) for it in node):
+        if node and all(isinstance(it, dict) and len(it) == 1 for it in node):
             merged: Dict[str, Any] = {}
             for it in node:
                 merged.update(it)

@@ -201,6 +201,12 @@ class ModelConfig(BaseConfig):
     seq_len_q: Optional[int] = opt(None, "unused")
     seq_len_kv: Optional[int] = opt(None, "unused")
     moe: MoEConfig = field(default_factory=MoEConfig)
+    layer_specs: Optional[List[dict]] = opt(None, "residual-stream families: one entry per layer, {type, mixer: sizes and "
+                                            "constants, mlp: {kind, ff} or null}")
+    layer_loop: Optional[dict] = opt(None, "residual-stream families: {start, stop, times}, the block "
+                                     "[start, stop) is evaluated `times` times, sharing its weights")
+    residual_streams: int = opt(1, "residual streams per token (hyper-connections)")
+    norm_groups: int = opt(1, "residual-stream families: equal parts of a row that are normed on their own")
     hf_model_type: Optional[str] = opt(None, "HuggingFace model_type")
     hf_architecture: Optional[str] = opt(None, "HuggingFace architecture name")
     tokenizer_type: str = opt("gpt2", "tokenizer type")

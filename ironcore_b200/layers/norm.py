@@ -48,6 +48,23 @@ class FusedRMSNorm(Norm):
         super().__init__(dim, eps, rms=True, bias=False, **kw)
 
 
+class GroupedRMSNorm(nn.Module):
+    """RMS norm over ``groups`` equal consecutive parts of a row, one gain per element (kept in fp32). The residual
+    stream boundary applies it; this module owns the parameters."""
+
+    def __init__(self, dim: int, groups: int, eps: float, device=None):
+        super().__init__()
+        if dim % groups:
+            raise ValueError(f"norm groups ({groups}) must divide the width ({dim})")
+        self.dim, self.groups, self.eps = dim, groups, float(eps)
+        self.layernorm = nn.Module()
+        self.layernorm.weight = nn.Parameter(torch.ones(dim, dtype=torch.float32, device=device))
+
+    @property
+    def weight(self) -> torch.Tensor:
+        return self.layernorm.weight
+
+
 def get_norm(config, dtype=None, device=None) -> Norm:
     m = config.model
     rms = m.ln_type == "rmsnorm"

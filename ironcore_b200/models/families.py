@@ -9,14 +9,15 @@ from __future__ import annotations
 
 import math
 
-FAMILIES = ("GPT", "LLAMA", "GEMMA1", "GEMMA", "QWEN", "PHI1", "PHI2", "MISTRAL", "MOE", "DUMMY")
+FAMILIES = ("GPT", "LLAMA", "GEMMA1", "GEMMA", "QWEN", "PHI1", "PHI2", "MISTRAL", "MOE", "DUMMY", "TETEPEL")
+STREAM_FAMILIES = ("TETEPEL",)      # several residual streams, layers listed in model.layer_specs
 
 
 def family_of(name: str) -> str:
     if not name:
         raise ValueError("model.name is required (e.g. gpt2-small, llama, gemma1, qwen, phi2, dummy)")
     up = name.upper().replace("-", "").replace("_", "")
-    for fam in ("GEMMA1", "GEMMA", "PHI1", "PHI2", "LLAMA", "QWEN", "MISTRAL", "GPT", "MOE", "DUMMY"):
+    for fam in ("GEMMA1", "GEMMA", "PHI1", "PHI2", "LLAMA", "QWEN", "MISTRAL", "GPT", "MOE", "DUMMY", "TETEPEL"):
         if up.startswith(fam):
             return "GEMMA1" if fam == "GEMMA" else fam
     raise ValueError(f"model '{name}' is not a supported family ({', '.join(FAMILIES)})")
@@ -27,6 +28,10 @@ def resolve_family_defaults(model_cfg) -> str:
     fam = family_of(model_cfg.name)
     m = model_cfg
     pe = m.positional_embedding
+    if fam in STREAM_FAMILIES:
+        pe.type, m.ln_type, m.no_bias = "none", "rmsnorm", True
+        if m.layer_specs:
+            m.num_layers = len(m.layer_specs)
     if m.qkv_bias is None:
         m.qkv_bias = True if fam == "QWEN" else (not m.no_bias)
     if m.norm_weight_offset is None:

@@ -20,12 +20,12 @@ import torch
 
 from ..layers.embedding import LanguageModelEmbedding
 from ..layers.module import BaseModule, init_parameters
-from ..layers.norm import get_norm
+from ..layers.norm import GroupedRMSNorm, get_norm
 from ..ops import functional as OF
 from ..parallel import collectives as C
 from ..parallel import mesh
 from ..parallel.tensor_parallel import ColumnParallelLinear, vocab_parallel_cross_entropy
-from .families import resolve_family_defaults
+from .families import STREAM_FAMILIES, resolve_family_defaults
 
 IGNORE_INDEX = -100
 
@@ -96,6 +96,12 @@ class LanguageModel(BaseModule):
             self.embedding = LanguageModelEmbedding(self.padded_vocab_size, self.vocab_size, m.d_model, m.max_seq_len,
                                                     False, 0.0, None, dtype, device)
             self.model = DummyModel(config, dtype, device)
+        elif self.family in STREAM_FAMILIES:
+            from .stream_model import StreamModel
+
+            self.model = StreamModel(config, dtype, device)
+            self.embedding = LanguageModelEmbedding(self.padded_vocab_size, self.vocab_size, self.model.width,
+                                                    max(m.max_seq_len, 1), False, 0.0, m.embed_scale, dtype, device)
         else:
             from .transformer import TransformerModel
 
@@ -103,7 +109,10 @@ class LanguageModel(BaseModule):
                                                     max(m.max_seq_len, 1), learned_pos, m.dropout_embd, m.embed_scale,
                                                     dtype, device)
             self.model = TransformerModel(config, dtype, device)
-        self.output_layernorm = get_norm(config, dtype, device)
+        if self.family in STREAM_FAMILIES:
+            self.output_layernorm = GroupedRMSNorm(m.d_model, m.norm_groups, m.ln_eps, device=device)
+        else:
+            self.output_layernorm = get_norm(config, dtype, device)
         self.untied = bool(m.untie_embed)
         if self.untied:
             self.output_layer = ColumnParallelLinear(m.d_model, self.padded_vocab_size, bias=bool(m.lm_head_bias),
@@ -125,6 +134,10 @@ class LanguageModel(BaseModule):
         if self.untied:
             self.output_layer.weight.vocab_valid = (1, self.vocab_size)
         init_parameters(self, self.config)
+        if self.family in STREAM_FAMILIES:
+            self.model.init_special()
+            with torch.no_grad():
+                self.embedding.word_embeddings.weight[:, self.model.d_model:].zero_()
         tp_rank = mesh.get_tensor_model_parallel_rank()
         # zero the padded vocabulary rows / columns
         with torch.no_grad():
@@ -180,6 +193,10 @@ class LanguageModel(BaseModule):
     def hidden_states(self, input_ids, position_ids=None, cu_seqlens=None, attn_mask=None):
         """[B, S] ids -> normalised final hidden states, token-major (SP shard when enabled)."""
         b, s = input_ids.shape
+        if self.family in STREAM_FAMILIES:
+            if position_ids is not None or cu_seqlens is not None or attn_mask is not None:
+                raise ValueError("residual-stream models take whole sequences: no positions, boundaries or masks")
+            return self._stream_hidden(input_ids), None
         if position_ids is None and cu_seqlens is None:
             position_ids, cu_seqlens = self._document_layout(input_ids)
         pos_flat = position_ids.reshape(-1).to(torch.int32) if position_ids is not None else None
@@ -187,6 +204,48 @@ class LanguageModel(BaseModule):
         x, aux = self.model(x, s, pos_flat, cu_seqlens, attn_mask)
         x = self.output_layernorm(x)
         return x, aux
+
+    # ------------------------------------------------------------------ residual-stream families
+    def step_hidden(self, batch, cache) -> torch.Tensor:
+        """Final-normed rows that ``batch`` asks for; ``cache`` is left with the batch's tokens in it."""
+        table = self.embedding.word_embeddings.weight
+        scale = 1.0 if self.embedding.scale is None else float(self.embedding.scale)
+        return self.model.hidden(batch, cache, table, scale, self.output_layernorm)
+
+    def step_logits(self, batch, cache) -> torch.Tensor:
+        """fp32 logits [rows, padded vocabulary] of the rows that ``batch`` asks for."""
+        from ..ops.latent import project
+
+        h = self.step_hidden(batch, cache)
+        if h.shape[0] == 0:
+            return torch.empty((0, self.padded_vocab_size), dtype=torch.float32, device=h.device)
+        return project(h, self.embedding.word_embeddings.weight, torch.float32)
+
+    def native_symbols(self):
+        """Entry points of the kernel library that serving this model calls (see ``ops.native.require``)."""
+        names = ["icb_stream_boundary", "icb_latent_norm"]
+        if self.dtype in (torch.bfloat16, torch.float16):
+            names += ["icb_gemm", "icb_gemm_2sm", "icb_glu_fwd", "icb_flash_fwd"]
+        return names if self.family in STREAM_FAMILIES else []
+
+    def _stream_hidden(self, input_ids: torch.Tensor) -> torch.Tensor:
+        """[B, S] ids -> final-normed rows [B * S, width], with a cache that lives for this call only."""
+        if torch.is_grad_enabled() and self.training:
+            raise NotImplementedError("residual-stream models have no backward pass: evaluate under torch.no_grad()")
+        from ..rl.batch import StepBatch
+
+        with torch.no_grad():
+            b, s = input_ids.shape
+            table = self.embedding.word_embeddings.weight
+            dev = table.device
+            cache = self.model.make_cache(b, s, 16, device=dev, dtype=table.dtype)
+            cache.reserve_all(b, s)
+            seqs = torch.arange(b, dtype=torch.int32, device=dev).repeat_interleave(s)
+            pos = torch.arange(s, dtype=torch.int32, device=dev).repeat(b)
+            cu = torch.arange(0, (b + 1) * s, s, dtype=torch.int32, device=dev)
+            batch = StepBatch(kind="prompt", tokens=input_ids.reshape(-1), seqs=seqs, positions=pos,
+                              slots=cache.slots_for(seqs, pos), max_len=s, max_context=s, cu_seqlens=cu, uniform=True)
+            return self.step_hidden(batch, cache)
 
     def logits_from_hidden(self, x: torch.Tensor) -> torch.Tensor:
         """token-major hidden [T(_local), d] -> vocab-sharded logits [T, V/t]."""

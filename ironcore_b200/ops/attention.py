@@ -12,7 +12,8 @@ from .native import call, dtype_code, ptr, stream_ptr
 
 native.register("icb_flash_fwd", [native.P] * 5 + [native.I, native.I, native.L, native.I, native.I, native.I,
                                                    native.L, native.L, native.P, native.I, native.F, native.I,
-                                                   native.P, native.P, native.F, native.P, native.I])
+                                                   native.P, native.P, native.F, native.P, native.I, native.I,
+                                                   native.P])
 native.register("icb_flash_bwd", [native.P] * 11 + [native.I, native.I, native.L, native.I, native.I, native.I,
                                                     native.L, native.L, native.L, native.L, native.P, native.I,
                                                     native.F, native.I, native.P, native.P, native.F, native.P])
@@ -101,8 +102,25 @@ def flash_fwd(qkv: torch.Tensor, hq: int, hkv: int, hd: int, seq_len: int, *, cu
     call("icb_flash_fwd", base, base + hq * hd * es, base + (hq + hkv) * hd * es, ptr(out), ptr(lse), batch, s, t,
          hq, hkv, hd, stride, stride, ptr(cu_seqlens), 1 if causal else 0, float(scale if scale else hd ** -0.5),
          dtype_code(qkv.dtype), ptr(native.status_tensor(qkv.device)), stream_ptr(), float(dropout_p),
-         ptr(dropout_seed), 1 if wide_tiles else 0)
+         ptr(dropout_seed), 1 if wide_tiles else 0, 0, None)
     return out, lse
+
+
+def flash_fwd_window(q: torch.Tensor, kv: torch.Tensor, heads: int, hd: int, cu_seqlens: torch.Tensor, max_seqlen: int,
+                     *, scale: float, window: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention of separate projections ``q`` [T, heads * hd] and ``kv`` [T, 2 * heads * hd] (keys, then
+    values) within the documents of ``cu_seqlens`` (int32 [n + 1], the longest being ``max_seqlen``). ``window`` > 0:
+    query i sees keys j with ``i - j < window``; key tiles outside are not visited. ``gate`` (fp32 [T, heads])
+    multiplies every head's output. Returns [T, heads * hd]."""
+    t = q.shape[0]
+    es = kv.element_size()
+    out = torch.empty((t, heads * hd), dtype=q.dtype, device=q.device)
+    lse = torch.empty((heads, t), dtype=torch.float32, device=q.device)
+    call("icb_flash_fwd", ptr(q), kv.data_ptr(), kv.data_ptr() + heads * hd * es, ptr(out), ptr(lse),
+         cu_seqlens.numel() - 1, int(max_seqlen), t, heads, heads, hd, q.stride(0), kv.stride(0), ptr(cu_seqlens), 1,
+         float(scale), dtype_code(q.dtype), ptr(native.status_tensor(q.device)), stream_ptr(), 0.0, None, 0,
+         int(window), ptr(gate))
+    return out
 
 
 def flash_bwd(dout: torch.Tensor, qkv: torch.Tensor, out: torch.Tensor, lse: torch.Tensor, hq: int, hkv: int, hd: int,

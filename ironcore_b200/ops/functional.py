@@ -197,6 +197,9 @@ def activation(x: torch.Tensor, name: str, row_limit: Optional[torch.Tensor] = N
     compute them; the other paths mask."""
     if name in GLU_KINDS:
         if use_native(x) and (x.shape[-1] // 2) % 8 == 0:
+            if not torch.is_grad_enabled() and x.dim() == 2 and x.stride(1) == 1 and x.stride(0) % 8 == 0 \
+                    and x.data_ptr() % 16 == 0:
+                return kernels.glu_fwd(x, name, row_limit)     # column slices are read in place
             return _Glu.apply(x.contiguous(), name, row_limit)
         note_fallback("gated activation", f"half width {x.shape[-1] // 2} is not a multiple of 8", x)
         if row_limit is not None:

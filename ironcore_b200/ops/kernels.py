@@ -151,7 +151,8 @@ def gemm(
         out_shape = (num_groups, m, n)
     else:
         out_shape = (m, n)
-    if out is None:
+    own_out = out is None
+    if own_out:
         out = torch.empty(out_shape, dtype=out_dtype, device=a.device)
     ldc = out.stride(-2)
     if out.stride(-1) != 1 or (ldc * out.element_size()) % 16 or out.data_ptr() % 16:
@@ -177,6 +178,8 @@ def gemm(
             call("icb_gemm_splitk", ptr(a), ptr(b), ptr(ws), ptr(bias), None, int(m), int(n), int(k), int(lda),
                  int(ldb), int(ws.stride(0)), 0, int(a_major), int(b_major), dtype_code(in_dt), int(split),
                  ptr(native.status_tensor(a.device)), stream_ptr())
+            if own_out and out_dtype == torch.float32 and residual is None:
+                return ws
             if n % 8 == 0 and out.dtype == in_dt and (residual is None or residual.dtype == in_dt):
                 call("icb_cast_add", ptr(ws), ptr(residual), ptr(out), int(m), int(n), int(ldr), int(ldc),
                      dtype_code(in_dt), stream_ptr())
@@ -298,13 +301,14 @@ def rope(x: torch.Tensor, out: torch.Tensor, *, nheads: int, head_dim: int, toke
 # ---------------------------------------------------------------------------
 def glu_fwd(x: torch.Tensor, name: str, row_limit: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``row_limit`` (int32 device tensor, one element): rows from that index on are not read and come out as
-    zeros (the unused capacity of a padded expert layout, which no kernel has written)."""
+    zeros (the unused capacity of a padded expert layout, which no kernel has written). A 2-D ``x`` may be a column
+    slice of a wider matrix."""
     kind, gate_is_act = GLU_KINDS[name]
     f = x.shape[-1] // 2
-    x2 = x.reshape(-1, 2 * f)
+    x2 = x if x.dim() == 2 and x.stride(1) == 1 else x.reshape(-1, 2 * f)
     y = torch.empty((x2.shape[0], f), dtype=x.dtype, device=x.device)
     call("icb_glu_fwd", ptr(x2), ptr(y), x2.shape[0], f, kind, gate_is_act, dtype_code(x.dtype), stream_ptr(),
-         ptr(row_limit))
+         ptr(row_limit), x2.stride(0))
     return y.view(*x.shape[:-1], f)
 
 

@@ -30,7 +30,7 @@ _SIGNATURES = {
     "icb_norm_fwd": [P, P, P, P, P, P, P, P, I, I, F, F, I, I, P, P],
     "icb_norm_bwd": [P, P, P, P, P, P, P, P, P, P, I, I, F, I, I, I, I, P, P],
     "icb_rope": [P, P, P, I, I, I, L, L, I, F, F, I, I, I, I, P, I],
-    "icb_glu_fwd": [P, P, L, I, I, I, I, P, P],
+    "icb_glu_fwd": [P, P, L, I, I, I, I, P, P, L],
     "icb_glu_bwd": [P, P, P, L, I, I, I, I, P, P],
     "icb_act_fwd": [P, P, L, I, I, P],
     "icb_act_bwd": [P, P, P, L, I, I, P],
@@ -56,6 +56,44 @@ def available() -> bool:
     return load(strict=True) is not None
 
 
+class _UnitLibrary:
+    """The entry points as attributes, from one shared library per source file, built when first asked for."""
+
+    def __init__(self):
+        from . import build as _build
+
+        self._build = _build
+        self._where = _build.exported_symbols()
+        self._libs = {}
+        self._lock = threading.Lock()
+
+    def require(self, names) -> None:
+        self._build.build_units(self._where[n] for n in names if n in self._where)
+
+    def __getattr__(self, name):
+        stem = self.__dict__["_where"].get(name)
+        if stem is None:
+            raise AttributeError(name)
+        with self._lock:
+            lib = self._libs.get(stem)
+            if lib is None:
+                lib = self._libs[stem] = C.CDLL(str(self._build.build_unit(stem)))
+        fn = getattr(lib, name)
+        if name in _SIGNATURES:
+            fn.argtypes = _SIGNATURES[name]
+        fn.restype = I
+        self.__dict__[name] = fn
+        return fn
+
+
+def require(names) -> None:
+    """Compile, side by side, whatever of the named entry points is not built yet (a checkout used for the first
+    time builds only what a model calls)."""
+    lib = load(strict=True)
+    if isinstance(lib, _UnitLibrary):
+        lib.require(names)
+
+
 def load(strict: bool = False):
     """Load (building if necessary) the native library. Returns None on CPU-only hosts
     unless ``strict``."""
@@ -65,11 +103,15 @@ def load(strict: bool = False):
     with _LOCK:
         if _LIB is not None:
             return _LIB
-        path = lib_path()
-        if not path.exists() or os.environ.get("ICB_REBUILD") == "1":
-            from . import build as _build
+        from . import build as _build
 
+        path = lib_path()
+        if os.environ.get("ICB_REBUILD") == "1":
             _build.build()
+        if not _build.is_current():
+            # never built, or built from other sources: the units are keyed by their sources and built on use
+            _LIB = _UnitLibrary()
+            return _LIB
         try:
             lib = C.CDLL(str(path))
         except OSError as exc:  # pragma: no cover - depends on host
@@ -90,7 +132,9 @@ def load(strict: bool = False):
 def register(name: str, argtypes) -> None:
     """Declare one more exported symbol (used by modules that own extra kernels)."""
     _SIGNATURES[name] = argtypes
-    if _LIB is not None:
+    if isinstance(_LIB, _UnitLibrary):
+        _LIB.__dict__.pop(name, None)
+    elif _LIB is not None:
         fn = getattr(_LIB, name, None)   # an optional entry point may be absent from an older build
         if fn is not None:
             fn.argtypes = argtypes

@@ -1,87 +1,109 @@
-"""Block (paged) KV cache: fixed-size pages, a host-side free list, per-sequence block tables.
+"""Paged caches: fixed-size pages, a host-side free list, per-sequence page tables.
 
-Per layer the cache holds ``k`` and ``v`` pools of shape ``[num_blocks, block_size, kv_heads, head_dim]``.
-A sequence owns a list of physical blocks; ``block_table[seq, i]`` is the block of its i-th page and
-``seq_lens[seq]`` its current length. The tables live on the device (updated in place, so a captured
-CUDA graph of the decode step keeps reading the current state)."""
+:class:`PagedCache` owns sequences and pages; what a page holds is up to the subclass. ``block_table[seq, i]`` is the
+physical block of a sequence's i-th page and ``seq_lens[seq]`` its current length; both live on the device and are
+updated in place, so a captured CUDA graph of the decode step keeps reading the current state.
+
+* :class:`BlockKVCache` — keys and values, pools ``[num_blocks, block_size, kv_heads, head_dim]`` per layer.
+* :class:`LatentCache` — one latent row per token and layer run, plus a fixed-size state per sequence and layer run."""
 
 from __future__ import annotations
 
-from typing import List
+from typing import Iterable, List, Optional, Sequence, Tuple
 
 import torch
 
 
-class BlockKVCache:
-    def __init__(self, num_layers: int, kv_heads: int, head_dim: int, num_blocks: int, block_size: int = 16,
-                 max_seqs: int = 128, max_seq_len: int = 1024, dtype=torch.bfloat16, device="cuda"):
+class PagedCache:
+    def __init__(self, num_blocks: int, block_size: int, max_seqs: int, max_seq_len: int, device):
         if block_size % 16:
             raise ValueError("block_size must be a multiple of 16")
-        self.num_layers, self.kv_heads, self.head_dim = num_layers, kv_heads, head_dim
         self.num_blocks, self.block_size = num_blocks, block_size
-        self.max_seqs = max_seqs
+        self.max_seqs, self.max_seq_len = max_seqs, max_seq_len
         self.max_blocks_per_seq = (max_seq_len + block_size - 1) // block_size
-        self.dtype, self.device = dtype, torch.device(device)
-        shape = (num_blocks, block_size, kv_heads, head_dim)
-        self.k = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
+        self.device = torch.device(device)
         self.block_table = torch.zeros((max_seqs, self.max_blocks_per_seq), dtype=torch.int32, device=self.device)
         self.seq_lens = torch.zeros(max_seqs, dtype=torch.int32, device=self.device)
-        self._free: List[int] = list(range(num_blocks - 1, -1, -1))
-        self._owned: List[List[int]] = [[] for _ in range(max_seqs)]
-        self._host_lens = [0] * max_seqs
+        self.reset()
 
-    # ---- allocation (host side) ----
+    # ---- sequences (host side) ----
+    def reset(self):
+        self._free: List[int] = list(range(self.num_blocks - 1, -1, -1))
+        self._owned: List[List[int]] = [[] for _ in range(self.max_seqs)]
+        self._dropped = [0] * self.max_seqs              # leading pages given back because no layer can see them
+        self._host_lens = [0] * self.max_seqs
+        self._idle: List[int] = list(range(self.max_seqs - 1, -1, -1))
+        self.seq_lens.zero_()
+
+    def acquire(self) -> int:
+        """A sequence number nobody uses."""
+        if not self._idle:
+            raise RuntimeError("all cache sequences are in use")
+        return self._idle.pop()
+
+    def release(self, seq: int):
+        """Give back a sequence obtained from :meth:`acquire` with everything it holds."""
+        self.free(seq)
+        self._idle.append(seq)
+
+    def length(self, seq: int) -> int:
+        return self._host_lens[seq]
+
+    def advance(self, seq: int, new_len: int):
+        """Host-side record of a sequence's length (``seq_lens`` is advanced by the step itself)."""
+        self._host_lens[seq] = new_len
+
+    # ---- pages (host side) ----
     @property
     def free_blocks(self) -> int:
         return len(self._free)
 
-    def reset(self):
-        self._free = list(range(self.num_blocks - 1, -1, -1))
-        self._owned = [[] for _ in range(self.max_seqs)]
-        self._host_lens = [0] * self.max_seqs
-        self.seq_lens.zero_()
-
     def reserve(self, seq: int, new_len: int):
         """Make sure sequence ``seq`` owns enough pages for ``new_len`` tokens."""
-        need = (new_len + self.block_size - 1) // self.block_size
-        owned = self._owned[seq]
-        if need > self.max_blocks_per_seq:
-            raise RuntimeError(f"sequence {seq} exceeds the cache's max_seq_len")
-        if need > len(owned):
-            add = need - len(owned)
-            if add > len(self._free):
-                raise RuntimeError("KV cache is out of blocks")
-            new = [self._free.pop() for _ in range(add)]
-            start = len(owned)
-            owned.extend(new)
-            self.block_table[seq, start:start + add] = torch.tensor(new, dtype=torch.int32, device=self.device)
+        self.reserve_many([(seq, new_len)])
 
     def reserve_all(self, num_seqs: int, new_len: int):
-        """Batched form of :meth:`reserve` for sequences 0..num_seqs-1 of equal length: one table write."""
-        need = (new_len + self.block_size - 1) // self.block_size
-        if need > self.max_blocks_per_seq:
-            raise RuntimeError("sequences exceed the cache's max_seq_len")
-        have = len(self._owned[0]) if num_seqs else 0
-        if any(len(self._owned[s]) != have for s in range(num_seqs)):
-            for s in range(num_seqs):
-                self.reserve(s, new_len)
-            return
-        add = need - have
-        if add <= 0:
-            return
-        if add * num_seqs > len(self._free):
+        """:meth:`reserve` for sequences 0..num_seqs-1."""
+        self.reserve_many([(s, new_len) for s in range(num_seqs)])
+
+    def reserve_many(self, wanted: Iterable[Tuple[int, int]]):
+        """:meth:`reserve` for several (sequence, length) pairs with one table update; all or nothing."""
+        plan = []
+        total = 0
+        for seq, new_len in wanted:
+            need = (new_len + self.block_size - 1) // self.block_size
+            if need > self.max_blocks_per_seq:
+                raise RuntimeError(f"sequence {seq} exceeds the cache's max_seq_len")
+            have = self._dropped[seq] + len(self._owned[seq])
+            if need > have:
+                plan.append((seq, have, need))
+                total += need - have
+        if total > len(self._free):
             raise RuntimeError("KV cache is out of blocks")
-        rows = []
-        for s in range(num_seqs):
-            new = [self._free.pop() for _ in range(add)]
-            self._owned[s].extend(new)
-            rows.append(new)
-        self.block_table[:num_seqs, have:have + add] = torch.tensor(rows, dtype=torch.int32, device=self.device)
+        rows, cols, blocks = [], [], []
+        for seq, have, need in plan:
+            for page in range(have, need):
+                blk = self._free.pop()
+                self._owned[seq].append(blk)
+                rows.append(seq)
+                cols.append(page)
+                blocks.append(blk)
+        if rows:
+            index = torch.tensor([rows, cols, blocks], dtype=torch.int64).to(self.device)
+            self.block_table[index[0], index[1]] = index[2].to(torch.int32)
+
+    def drop_before(self, seq: int, position: int):
+        """Give back the pages of ``seq`` that end at or before ``position`` (no later token sees them)."""
+        n = position // self.block_size - self._dropped[seq]
+        if n > 0:
+            self._free.extend(reversed(self._owned[seq][:n]))
+            del self._owned[seq][:n]
+            self._dropped[seq] += n
 
     def free(self, seq: int):
         self._free.extend(reversed(self._owned[seq]))
         self._owned[seq] = []
+        self._dropped[seq] = 0
         self._host_lens[seq] = 0
         self.seq_lens[seq] = 0
 
@@ -92,5 +114,44 @@ class BlockKVCache:
         blk = self.block_table[seq_ids.long(), page].long()
         return blk * self.block_size + (positions % self.block_size).long()
 
+    @property
+    def window(self) -> int:
+        """The furthest any layer looks back, the token itself included; 0 = to the first token."""
+        return 0
+
+
+class BlockKVCache(PagedCache):
+    def __init__(self, num_layers: int, kv_heads: int, head_dim: int, num_blocks: int, block_size: int = 16,
+                 max_seqs: int = 128, max_seq_len: int = 1024, dtype=torch.bfloat16, device="cuda"):
+        super().__init__(num_blocks, block_size, max_seqs, max_seq_len, device)
+        self.num_layers, self.kv_heads, self.head_dim, self.dtype = num_layers, kv_heads, head_dim, dtype
+        shape = (num_blocks, block_size, kv_heads, head_dim)
+        self.k = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
+        self.v = [torch.zeros(shape, dtype=dtype, device=self.device) for _ in range(num_layers)]
+
     def bytes_per_token(self) -> int:
         return 2 * self.num_layers * self.kv_heads * self.head_dim * torch.empty((), dtype=self.dtype).element_size()
+
+
+class LatentCache(PagedCache):
+    """``latent[run]``: rows [num_blocks * block_size, row width of that run]. ``shift_state[run]``: fp32
+    [max_seqs, state width], the last normed input of every sequence. With a ``window``, pages that no layer can see
+    any more go back to the free list while a sequence is still running."""
+
+    def __init__(self, row_widths: Sequence[int], state_width: int, *, max_seqs: int, max_seq_len: int,
+                 block_size: int = 16, num_blocks: Optional[int] = None, window: int = 0, dtype=torch.bfloat16,
+                 device="cuda"):
+        if num_blocks is None:
+            num_blocks = max_seqs * ((max_seq_len + block_size - 1) // block_size)
+        super().__init__(num_blocks, block_size, max_seqs, max_seq_len, device)
+        self._window, self.dtype, self.row_widths = int(window), dtype, list(row_widths)
+        self.latent = [torch.zeros((num_blocks * block_size, w), dtype=dtype, device=self.device) for w in row_widths]
+        self.shift_state = [torch.zeros((max_seqs, state_width), dtype=torch.float32, device=self.device)
+                            for _ in row_widths]
+
+    @property
+    def window(self) -> int:
+        return self._window
+
+    def bytes_per_token(self) -> int:
+        return sum(self.row_widths) * torch.empty((), dtype=self.dtype).element_size()
