@@ -88,7 +88,7 @@ __device__ __forceinline__ float act_f(int kind, float x) {
     case 1: return 0.5f * x * (1.f + erff(x * 0.70710678118654752f));
     case 2: {
       const float u = 0.7978845608028654f * (x + 0.044715f * x * x * x);
-      return 0.5f * x * (1.f + tanhf(u));
+      return __fdividef(x, 1.f + __expf(-2.f * u));      // 0.5 x (1 + tanh u) = x sigmoid(2 u)
     }
     case 3: return __fdividef(x, 1.f + __expf(-x));
     default: return __fdividef(1.f, 1.f + __expf(-x));

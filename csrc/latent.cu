@@ -8,10 +8,10 @@
 //                         latents, writes the latent to its cache row, and the sigmoid of the gates.
 //  * head_product       : out[t, n, :] = B_n a[t, n, :] (optionally times a gate per (t, n)): the query-side and
 //                         output-side products, one small matrix per head, weights streamed once.
-//  * latent_attend_mma  : tensor-core attention of single query rows, 16 heads per CTA. Latent rows come in tiles of
-//                         32 tokens by cp.async, double or triple buffered; a tile is both K and V. The eight warps
-//                         split S = Q C^T over (token group, half of the rank) and O += P C over rank columns. The
-//                         visible range can be cut over CTAs, with latent_merge joining the parts.
+//  * latent_attend_mma  : tensor-core attention of single query rows, 16 or 32 heads per CTA. Latent rows come in tiles
+//                         of 32 tokens by cp.async, double or triple buffered; a tile is both K and V. Four warps own
+//                         a quarter of the rank columns each. The visible range can be cut over CTAs, with
+//                         latent_merge joining the parts.
 //  * latent_attend_rows : the same for any rank and type on plain FMAs (fp32 models, ranks beyond 512).
 // A query row is (sequence slot, position): its keys are the `window` tokens that end with itself (window <= 0: all up to itself), so
 // decoding, continued prompts and mixed batches are the same call.
@@ -25,42 +25,102 @@ namespace icb {
 constexpr int kLatentNormThreads = 128;
 
 template <typename T>
+__device__ __forceinline__ void store4(T* p, float a, float b, float c, float d);
+template <>
+__device__ __forceinline__ void store4<float>(float* p, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+template <>
+__device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float a, float b, float c, float d) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(a, b), pack_bf16x2(c, d));
+}
+
+// WPR warps per row: 1 for many rows (no block-wide step), 4 for a few. VEC 4 needs q_rank, rank, ldq and rp to be
+// multiples of 4 (ldz always is).
+template <typename T, int WPR, int VEC>
 __global__ void __launch_bounds__(kLatentNormThreads)
 latent_norm_kernel(const float* __restrict__ z, long long ldz, const float* __restrict__ wq,
                    const float* __restrict__ wc, T* __restrict__ cq, int ldq, T* __restrict__ c,
                    T* __restrict__ cache, const long long* __restrict__ slots, float* __restrict__ gate, int rows,
                    int q_rank, int rank, int rp, int heads, float eps) {
+  constexpr int kRowsPerBlock = kLatentNormThreads / 32 / WPR;
+  constexpr int kStep = WPR * 32 * VEC;
   __shared__ float red[2][kLatentNormThreads / 32];
-  const int row = blockIdx.x;
-  if (row >= rows) return;
+  const int row = blockIdx.x * kRowsPerBlock + (WPR == 1 ? threadIdx.x >> 5 : 0);
+  const int first = (WPR == 1 ? threadIdx.x & 31 : threadIdx.x) * VEC;
+  if (row >= rows) return;                               // whole warps (WPR 1) or whole blocks
   const float* zq = z + (size_t)row * ldz;
   const float* zc = zq + q_rank;
   const float* zg = zc + rank;
-  float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x; i < q_rank; i += kLatentNormThreads) sq += zq[i] * zq[i];
-  for (int i = threadIdx.x; i < rank; i += kLatentNormThreads) sc += zc[i] * zc[i];
-  sq = warp_sum(sq);
-  sc = warp_sum(sc);
-  if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sc; }
-  __syncthreads();
-  sq = sc = 0.f;
+  auto square_sum = [&](const float* p, int n) {
+    float s = 0.f;
+#pragma unroll 4
+    for (int i = first; i < n; i += kStep) {
+      if constexpr (VEC == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p + i);
+        s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      } else {
+        s += p[i] * p[i];
+      }
+    }
+    return warp_sum(s);
+  };
+  float sq = square_sum(zq, q_rank), sc = square_sum(zc, rank);
+  if constexpr (WPR > 1) {
+    if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sc; }
+    __syncthreads();
+    sq = sc = 0.f;
 #pragma unroll
-  for (int w = 0; w < kLatentNormThreads / 32; ++w) { sq += red[0][w]; sc += red[1][w]; }
+    for (int w = 0; w < WPR; ++w) { sq += red[0][w]; sc += red[1][w]; }
+  }
   const float iq = 1.f / sqrtf(sq / (float)q_rank + eps);
   const float ic = 1.f / sqrtf(sc / (float)rank + eps);
-  T* q_row = cq + (size_t)row * ldq;
-  for (int i = threadIdx.x; i < ldq; i += kLatentNormThreads)
-    q_row[i] = static_cast<T>(i < q_rank ? zq[i] * iq * wq[i] : 0.f);
+  // scaled row with a zero tail up to `width`, to one or two destinations
+  auto emit = [&](const float* p, const float* w, float inv, int n, int width, T* d0, T* d1) {
+#pragma unroll 4
+    for (int i = first; i < width; i += kStep) {
+      if constexpr (VEC == 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n) {
+          const float4 x = *reinterpret_cast<const float4*>(p + i);
+          const float4 g = *reinterpret_cast<const float4*>(w + i);
+          v = make_float4(x.x * inv * g.x, x.y * inv * g.y, x.z * inv * g.z, x.w * inv * g.w);
+        }
+        if (d0 != nullptr) store4<T>(d0 + i, v.x, v.y, v.z, v.w);
+        if (d1 != nullptr) store4<T>(d1 + i, v.x, v.y, v.z, v.w);
+      } else {
+        const T v = static_cast<T>(i < n ? p[i] * inv * w[i] : 0.f);
+        if (d0 != nullptr) d0[i] = v;
+        if (d1 != nullptr) d1[i] = v;
+      }
+    }
+  };
+  emit(zq, wq, iq, q_rank, ldq, cq + (size_t)row * ldq, nullptr);
   const long long slot = cache != nullptr ? slots[row] : -1;
-  T* cache_row = slot >= 0 ? cache + (size_t)slot * rp : nullptr;
-  T* c_row = c != nullptr ? c + (size_t)row * rp : nullptr;
-  for (int i = threadIdx.x; i < rp; i += kLatentNormThreads) {
-    const T v = static_cast<T>(i < rank ? zc[i] * ic * wc[i] : 0.f);
-    if (cache_row != nullptr) cache_row[i] = v;
-    if (c_row != nullptr) c_row[i] = v;
-  }
-  for (int i = threadIdx.x; i < heads; i += kLatentNormThreads)
+  emit(zc, wc, ic, rank, rp, slot >= 0 ? cache + (size_t)slot * rp : nullptr,
+       c != nullptr ? c + (size_t)row * rp : nullptr);
+  for (int i = first / VEC; i < heads; i += WPR * 32)
     gate[(size_t)row * heads + i] = 1.f / (1.f + expf(-zg[i]));
+}
+
+template <typename T>
+static int launch_latent_norm(const float* z, long long ldz, const float* wq, const float* wc, void* cq, int ldq,
+                              void* c, void* cache, const long long* slots, float* gate, int rows, int q_rank, int rank,
+                              int rp, int heads, float eps, cudaStream_t st) {
+  const bool wide = q_rank % 4 == 0 && rank % 4 == 0 && ldq % 4 == 0 && rp % 4 == 0 && ldz % 4 == 0;
+#define ICB_LN(WPR, VEC)                                                                                              \
+  latent_norm_kernel<T, WPR, VEC><<<WPR == 1 ? (rows + 3) / 4 : rows, kLatentNormThreads, 0, st>>>(                   \
+      z, ldz, wq, wc, reinterpret_cast<T*>(cq), ldq, reinterpret_cast<T*>(c), reinterpret_cast<T*>(cache), slots, gate, \
+      rows, q_rank, rank, rp, heads, eps)
+  if (rows >= 8 * num_sms()) {
+    if (wide) ICB_LN(1, 4);
+    else ICB_LN(1, 1);
+  } else {
+    if (wide) ICB_LN(4, 4);
+    else ICB_LN(4, 1);
+  }
+#undef ICB_LN
+  return check_launch("latent_norm_kernel");
 }
 
 // ----------------------------------------------------------------------------------------------- head_product
@@ -227,7 +287,8 @@ __global__ void __launch_bounds__(kLrChunk) latent_attend_rows_kernel(const Late
 }
 
 // ------------------------------------------------------------------------------------------ latent_attend_mma
-constexpr int kLmThreads = 256;
+constexpr int kLmThreads = 128;
+constexpr int kLmWarps = kLmThreads / 32;
 constexpr int kLmTok = 32;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -246,37 +307,39 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-template <int NT>   // rp = 64 * NT
+template <int NT, int MT>   // rp = 64 * NT, MT * 16 heads per CTA
 struct LmSmem {
   static constexpr int kRp = 64 * NT;
   static constexpr int kPitch = kRp + 8;                   // rows 16 bytes apart modulo 128: ldmatrix without conflicts
   static constexpr int kStages = NT <= 4 ? 3 : 2;
-  static constexpr int q_bytes = 16 * kPitch * 2;
   static constexpr int tile_bytes = kLmTok * kPitch * 2;
-  static constexpr int s_off = q_bytes + kStages * tile_bytes;
-  static constexpr int kSPitch = kLmTok + 1;
-  static constexpr int s_bytes = 2 * 16 * kSPitch * 4;
+  static constexpr int s_off = kStages * tile_bytes;
+  static constexpr int kSPitch = kLmTok + 8;               // float pairs of a fragment row land in distinct banks
+  static constexpr int s_bytes = kLmWarps * MT * 16 * kSPitch * 4;
   static constexpr int p_off = s_off + s_bytes;
   static constexpr int kPPitch = kLmTok + 8;
-  static constexpr int p_bytes = 16 * kPPitch * 2;
-  static constexpr int row_off = p_off + p_bytes;          // corr, m, l: 16 floats each
-  static constexpr int total = row_off + 3 * 16 * 4;
+  static constexpr int p_bytes = MT * 16 * kPPitch * 2;
+  static constexpr int row_off = p_off + p_bytes;          // corr, m, l: MT * 16 floats each
+  static constexpr int total = row_off + 3 * MT * 16 * 4;
 };
 
-template <int NT>
+// A warp owns a quarter of the rank columns in both products. Its slice of Q stays in registers; S = Q C^T is the sum
+// of the four slices' parts, which meet in shared memory; O += P C needs nothing from the other warps but P.
+template <int NT, int MT>
 __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const LatentAttendArgs a) {
-  using L = LmSmem<NT>;
+  using L = LmSmem<NT, MT>;
+  constexpr int kRows = MT * 16;
   extern __shared__ __align__(128) uint8_t lm_smem[];
-  const int row = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
+  const int row = blockIdx.x, h0 = blockIdx.y * kRows, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int fr = lane >> 2, fc = lane & 3;                   // fragment row / column pair of this lane
   float* sS = reinterpret_cast<float*>(lm_smem + L::s_off);
   __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(lm_smem + L::p_off);
   float* s_corr = reinterpret_cast<float*>(lm_smem + L::row_off);
-  float* s_m = s_corr + 16;
-  float* s_l = s_corr + 32;
-  const uint32_t q_addr = smem_u32(lm_smem);
-  const uint32_t c_addr = q_addr + L::q_bytes;
-  const uint32_t p_addr = q_addr + L::p_off;
+  float* s_m = s_corr + kRows;
+  float* s_l = s_m + kRows;
+  const uint32_t c_addr = smem_u32(lm_smem);
+  const uint32_t p_addr = c_addr + L::p_off;
 
   const int pos = a.row_pos[row];
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
@@ -286,29 +349,25 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
   const int* bt = a.block_table + (size_t)a.row_seq[row] * a.max_blocks;
   const uint16_t* cache = reinterpret_cast<const uint16_t*>(a.cache);
 
-  {
-    const uint16_t* q = reinterpret_cast<const uint16_t*>(a.q) + (size_t)row * a.heads * L::kRp;
-    for (int i = threadIdx.x; i < 16 * (L::kRp / 8); i += kLmThreads) {
-      const int hr = i / (L::kRp / 8), ch = i - hr * (L::kRp / 8);
-      const bool ok = h0 + hr < a.heads;
-      cp_async16(q_addr + hr * (L::kPitch * 2) + ch * 16, q + (size_t)(ok ? h0 + hr : 0) * L::kRp + ch * 8, ok);
-    }
-  }
-  auto load_tile = [&](int t) {                              // eight threads per token row
+  auto load_tile = [&](int t) {                              // eight threads per token row, sixteen rows at a time
     if (t < t_end) {
-      const int tr = threadIdx.x >> 3;
-      const int tok = lo + t * kLmTok + tr;
-      const bool ok = tok <= pos;
-      const uint16_t* src = cache;
-      if (ok) {
-        const int page = tok / a.block_size;
-        src = cache + ((size_t)bt[page] * a.block_size + (tok - page * a.block_size)) * L::kRp;
-      }
-      const uint32_t dst = c_addr + ((t - t_begin) % L::kStages) * L::tile_bytes + tr * (L::kPitch * 2);
+      const uint32_t stage = c_addr + ((t - t_begin) % L::kStages) * L::tile_bytes;
 #pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        const int ch = (threadIdx.x & 7) + j * 8;
-        cp_async16(dst + ch * 16, src + ch * 8, ok);
+      for (int half = 0; half < 2; ++half) {
+        const int tr = (threadIdx.x >> 3) + half * 16;
+        const int tok = lo + t * kLmTok + tr;
+        const bool ok = tok <= pos;
+        const uint16_t* src = cache;
+        if (ok) {
+          const int page = tok / a.block_size;
+          src = cache + ((size_t)bt[page] * a.block_size + (tok - page * a.block_size)) * L::kRp;
+        }
+        const uint32_t dst = stage + tr * (L::kPitch * 2);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          const int ch = (threadIdx.x & 7) + j * 8;
+          cp_async16(dst + ch * 16, src + ch * 8, ok);
+        }
       }
     }
     cp_async_commit();
@@ -316,100 +375,154 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
 #pragma unroll
   for (int s = 0; s < L::kStages - 1; ++s) load_tile(t_begin + s);
 
-  float acc[NT][4];
+  const int col0 = warp * (16 * NT);                         // this warp's rank columns
+  uint32_t qf[MT][NT][4];
+  {
+    const uint16_t* q = reinterpret_cast<const uint16_t*>(a.q) + (size_t)row * a.heads * L::kRp + col0 + 2 * fc;
 #pragma unroll
-  for (int n = 0; n < NT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};    // of rows 2 warp, 2 warp + 1, the same in every lane
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int k = 0; k < NT; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int hr = h0 + mt * 16 + fr + (e & 1) * 8;
+          qf[mt][k][e] = hr < a.heads
+              ? *reinterpret_cast<const uint32_t*>(q + (size_t)hr * L::kRp + k * 16 + (e >> 1) * 8) : 0u;
+        }
+  }
+  float acc[MT][2 * NT][4];
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int n = 0; n < 2 * NT; ++n) acc[mt][n][0] = acc[mt][n][1] = acc[mt][n][2] = acc[mt][n][3] = 0.f;
+  constexpr int kOwn = kRows / kLmWarps;                     // heads whose softmax this warp does
+  float m[kOwn], l[kOwn];                                    // m: the same in every lane; l: this lane's share
+#pragma unroll
+  for (int e = 0; e < kOwn; ++e) { m[e] = -INFINITY; l[e] = 0.f; }
   const float scale_log2 = a.scale * 1.4426950408889634f;
-  const int tg = warp & 3, kh = warp >> 2;                   // token group and rank half of this warp's scores
+  const uint32_t s_lane = (((lane >> 4) * 8 + (lane & 7)) * L::kPitch + ((lane >> 3) & 1) * 8 + col0) * 2;
+  const uint32_t v_lane = (lane * L::kPitch + col0) * 2;
 
   for (int t = t_begin; t < t_end; ++t) {
     cp_async_wait<L::kStages - 2>();
     __syncthreads();                                         // tile t is in place, everybody is done with tile t - 1
     load_tile(t + L::kStages - 1);
     const uint32_t tile = c_addr + ((t - t_begin) % L::kStages) * L::tile_bytes;
-    // ---- scores: 16 heads x 8 tokens over half of the rank, two k-steps per round
-    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-    for (int i = 0; i < NT; ++i) {
-      const int k0 = kh * (L::kRp / 2) + i * 32;
-      uint32_t b[4], a0[4], a1[4];
-      ldsm_x4(b, tile + (tg * 8 + (lane & 7)) * (L::kPitch * 2) + (k0 + (lane >> 3) * 8) * 2);
-      const uint32_t qa = q_addr + (lane & 15) * (L::kPitch * 2) + (k0 + (lane >> 4) * 8) * 2;
-      ldsm_x4(a0, qa);
-      ldsm_x4(a1, qa + 32);
-      mma_bf16_16816(s0, a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
-      mma_bf16_16816(s1, a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
-    }
+    // ---- this slice's part of the scores, heads x 32 tokens
     {
-      float* dst = sS + kh * 16 * L::kSPitch + tg * 8 + 2 * (lane & 3);
-      const int r = lane >> 2;
-      dst[r * L::kSPitch] = s0[0] + s1[0];
-      dst[r * L::kSPitch + 1] = s0[1] + s1[1];
-      dst[(r + 8) * L::kSPitch] = s0[2] + s1[2];
-      dst[(r + 8) * L::kSPitch + 1] = s0[3] + s1[3];
+      float sc[MT][4][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int n = 0; n < 4; ++n) sc[mt][n][0] = sc[mt][n][1] = sc[mt][n][2] = sc[mt][n][3] = 0.f;
+#pragma unroll
+      for (int k = 0; k < NT; ++k) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          uint32_t b[4];
+          ldsm_x4(b, tile + s_lane + half * 16 * (L::kPitch * 2) + k * 32);
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            mma_bf16_16816(sc[mt][2 * half], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[0], b[1]);
+            mma_bf16_16816(sc[mt][2 * half + 1], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[2], b[3]);
+          }
+        }
+      }
+      float* dst = sS + (warp * kRows + fr) * L::kSPitch + 2 * fc;
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          float* d = dst + mt * 16 * L::kSPitch + n * 8;
+          *reinterpret_cast<float2*>(d) = make_float2(sc[mt][n][0], sc[mt][n][1]);
+          *reinterpret_cast<float2*>(d + 8 * L::kSPitch) = make_float2(sc[mt][n][2], sc[mt][n][3]);
+        }
     }
     __syncthreads();
-    // ---- online softmax: warp w owns heads 2w, 2w + 1; a lane is a token of the tile (the first one is always visible)
-    const bool seen = lo + t * kLmTok + lane <= pos;
+    // ---- online softmax of this warp's heads; a lane is a token of the tile (the first one is always visible)
+    {
+      const bool seen = lo + t * kLmTok + lane <= pos;
+      float s[kOwn], mx[kOwn];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int hr = warp * 2 + e;
-      const float s = seen ? (sS[hr * L::kSPitch + lane] + sS[(16 + hr) * L::kSPitch + lane]) * scale_log2 : -INFINITY;
-      float mx = s;
+      for (int e = 0; e < kOwn; ++e) {
+        float v = 0.f;
 #pragma unroll
-      for (int off = 16; off; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      mx = fmaxf(mx, m[e]);
-      const float corr = exp2f(m[e] - mx);
-      const float p = exp2f(s - mx);
-      l[e] = l[e] * corr + warp_sum(p);
-      m[e] = mx;
-      sP[hr * L::kPPitch + lane] = __float2bfloat16(p);
-      if (lane == 0) s_corr[hr] = corr;
+        for (int w = 0; w < kLmWarps; ++w) v += sS[(w * kRows + warp * kOwn + e) * L::kSPitch + lane];
+        s[e] = mx[e] = seen ? v * scale_log2 : -INFINITY;
+      }
+#pragma unroll
+      for (int off = 16; off; off >>= 1)
+#pragma unroll
+        for (int e = 0; e < kOwn; ++e) mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], off));
+#pragma unroll
+      for (int e = 0; e < kOwn; ++e) {
+        const float top = fmaxf(mx[e], m[e]);
+        const float corr = exp2f(m[e] - top);
+        const float p = exp2f(s[e] - top);
+        l[e] = l[e] * corr + p;
+        m[e] = top;
+        sP[(warp * kOwn + e) * L::kPPitch + lane] = __float2bfloat16(p);
+        if (lane == 0) s_corr[warp * kOwn + e] = corr;
+      }
     }
     __syncthreads();
-    // ---- O = O * corr + P C over this warp's rank columns
-    const float c0 = s_corr[lane >> 2], c1 = s_corr[(lane >> 2) + 8];
-    uint32_t pa[4], pb[4];
-    const uint32_t pl = p_addr + (lane & 15) * (L::kPPitch * 2) + (lane >> 4) * 16;
-    ldsm_x4(pa, pl);
-    ldsm_x4(pb, pl + 32);
+    // ---- O = O * corr + P C over this warp's columns
+    uint32_t pa[MT][2][4];
 #pragma unroll
-    for (int n = 0; n < NT; ++n) {
+    for (int mt = 0; mt < MT; ++mt) {
+      const uint32_t pl = p_addr + ((mt * 16 + (lane & 15)) * L::kPPitch + (lane >> 4) * 8) * 2;
+      ldsm_x4(pa[mt][0], pl);
+      ldsm_x4(pa[mt][1], pl + 32);
+      const float c0 = s_corr[mt * 16 + fr], c1 = s_corr[mt * 16 + fr + 8];
+      if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
+#pragma unroll
+        for (int n = 0; n < 2 * NT; ++n) {
+          acc[mt][n][0] *= c0; acc[mt][n][1] *= c0; acc[mt][n][2] *= c1; acc[mt][n][3] *= c1;
+        }
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 2 * NT; ++n) {
       uint32_t b[4];
-      ldsm_x4_t(b, tile + lane * (L::kPitch * 2) + (warp * (8 * NT) + n * 8) * 2);
-      acc[n][0] *= c0; acc[n][1] *= c0; acc[n][2] *= c1; acc[n][3] *= c1;
-      mma_bf16_16816(acc[n], pa[0], pa[1], pa[2], pa[3], b[0], b[1]);
-      mma_bf16_16816(acc[n], pb[0], pb[1], pb[2], pb[3], b[2], b[3]);
-    }
-  }
-  cp_async_wait<0>();
-  if (lane < 2) {
-    s_m[warp * 2 + lane] = lane ? m[1] : m[0];
-    s_l[warp * 2 + lane] = lane ? l[1] : l[0];
-  }
-  __syncthreads();
+      ldsm_x4_t(b, tile + v_lane + n * 16);
 #pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const int hr = (lane >> 2) + half * 8;
-    if (h0 + hr < a.heads) {
-      const int col = warp * (8 * NT) + 2 * (lane & 3);
-      const size_t head_row = (size_t)row * a.heads + h0 + hr;
-      if (a.nsplit == 1) {
-        const float inv = s_l[hr] > 0.f ? 1.f / s_l[hr] : 0.f;
-        uint16_t* o = reinterpret_cast<uint16_t*>(a.out) + head_row * L::kRp + col;
-#pragma unroll
-        for (int n = 0; n < NT; ++n)
-          *reinterpret_cast<uint32_t*>(o + n * 8) = pack_bf16x2(acc[n][half * 2] * inv, acc[n][half * 2 + 1] * inv);
-      } else {
-        float* rec = a.part + (head_row * a.nsplit + split) * (L::kRp + 2);
-#pragma unroll
-        for (int n = 0; n < NT; ++n)
-          *reinterpret_cast<float2*>(rec + col + n * 8) = make_float2(acc[n][half * 2], acc[n][half * 2 + 1]);
-        if (warp == 0 && (lane & 3) == 0) *reinterpret_cast<float2*>(rec + L::kRp) = make_float2(s_m[hr], s_l[hr]);
+      for (int mt = 0; mt < MT; ++mt) {
+        mma_bf16_16816(acc[mt][n], pa[mt][0][0], pa[mt][0][1], pa[mt][0][2], pa[mt][0][3], b[0], b[1]);
+        mma_bf16_16816(acc[mt][n], pa[mt][1][0], pa[mt][1][1], pa[mt][1][2], pa[mt][1][3], b[2], b[3]);
       }
     }
   }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int e = 0; e < kOwn; ++e) {
+    const float sum = warp_sum(l[e]);
+    if (lane == 0) { s_m[warp * kOwn + e] = m[e]; s_l[warp * kOwn + e] = sum; }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int hr = mt * 16 + fr + half * 8;
+      if (h0 + hr < a.heads) {
+        const int col = col0 + 2 * fc;
+        const size_t head_row = (size_t)row * a.heads + h0 + hr;
+        if (a.nsplit == 1) {
+          const float inv = s_l[hr] > 0.f ? 1.f / s_l[hr] : 0.f;
+          uint16_t* o = reinterpret_cast<uint16_t*>(a.out) + head_row * L::kRp + col;
+#pragma unroll
+          for (int n = 0; n < 2 * NT; ++n)
+            *reinterpret_cast<uint32_t*>(o + n * 8) =
+                pack_bf16x2(acc[mt][n][half * 2] * inv, acc[mt][n][half * 2 + 1] * inv);
+        } else {
+          float* rec = a.part + (head_row * a.nsplit + split) * (L::kRp + 2);
+#pragma unroll
+          for (int n = 0; n < 2 * NT; ++n)
+            *reinterpret_cast<float2*>(rec + col + n * 8) = make_float2(acc[mt][n][half * 2], acc[mt][n][half * 2 + 1]);
+          if (warp == 0 && fc == 0) *reinterpret_cast<float2*>(rec + L::kRp) = make_float2(s_m[hr], s_l[hr]);
+        }
+      }
+    }
 }
 
 // Joins the parts of one (row, head): running maxima are in the log2 domain; an empty part has max -inf and sum 0.
@@ -434,18 +547,22 @@ latent_merge_kernel(const float* __restrict__ part, uint16_t* __restrict__ out, 
   }
 }
 
-template <int NT>
-static int launch_latent_mma(const LatentAttendArgs& a, cudaStream_t st) {
-  auto kern = latent_attend_mma_kernel<NT>;
+template <int NT, int MT>
+static int launch_latent_mma_m(const LatentAttendArgs& a, cudaStream_t st) {
+  auto kern = latent_attend_mma_kernel<NT, MT>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, LmSmem<NT>::total);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, LmSmem<NT, MT>::total);
     if (e != cudaSuccess) return -(int)e;
     configured = true;
   }
-  dim3 grid(a.rows, (a.heads + 15) / 16, a.nsplit);
-  kern<<<grid, kLmThreads, LmSmem<NT>::total, st>>>(a);
+  dim3 grid(a.rows, (a.heads + MT * 16 - 1) / (MT * 16), a.nsplit);
+  kern<<<grid, kLmThreads, LmSmem<NT, MT>::total, st>>>(a);
   return check_launch("latent_attend_mma_kernel");
+}
+template <int NT>
+static int launch_latent_mma(const LatentAttendArgs& a, cudaStream_t st) {
+  return a.heads > 16 ? launch_latent_mma_m<NT, 2>(a, st) : launch_latent_mma_m<NT, 1>(a, st);
 }
 
 }  // namespace icb
@@ -462,16 +579,12 @@ ICB_API int icb_latent_norm(const float* z, long long ldz, const float* wq, cons
   if (cache != nullptr && slots == nullptr) return -4;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == kBF16)
-    latent_norm_kernel<__nv_bfloat16><<<rows, kLatentNormThreads, 0, st>>>(
-        z, ldz, wq, wc, reinterpret_cast<__nv_bfloat16*>(cq), ldq, reinterpret_cast<__nv_bfloat16*>(c),
-        reinterpret_cast<__nv_bfloat16*>(cache), slots, gate, rows, q_rank, rank, rp, heads, eps);
-  else if (dtype == kF32)
-    latent_norm_kernel<float><<<rows, kLatentNormThreads, 0, st>>>(
-        z, ldz, wq, wc, reinterpret_cast<float*>(cq), ldq, reinterpret_cast<float*>(c), reinterpret_cast<float*>(cache),
-        slots, gate, rows, q_rank, rank, rp, heads, eps);
-  else
-    return -3;
-  return check_launch("latent_norm_kernel");
+    return launch_latent_norm<__nv_bfloat16>(z, ldz, wq, wc, cq, ldq, c, cache, slots, gate, rows, q_rank, rank, rp,
+                                             heads, eps, st);
+  if (dtype == kF32)
+    return launch_latent_norm<float>(z, ldz, wq, wc, cq, ldq, c, cache, slots, gate, rows, q_rank, rank, rp, heads, eps,
+                                     st);
+  return -3;
 }
 
 // out[rows, heads, N] = per head: a[rows, heads, K] B[heads, N, K]^T (times gate[rows, heads] when given).

@@ -284,13 +284,15 @@ ICB_API int icb_stream_boundary(const long long* tokens, const void* table, long
   a.row_seq = row_seq; a.row_pos = row_pos; a.T = T; a.S = S; a.D = D;
   const int gs = D / groups;
   const bool wide = D % 4 == 0 && gs % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0 && ldr % 4 == 0 && ld_table % 4 == 0;
-  // about 8 warps: a whole number per group, but no more than a group has vectors for
+  // about 8 warps (16 when there are only a few rows, where latency counts): a whole number per group, but no more
+  // than a group has vectors for
+  const int target = T <= 2 * num_sms() ? 16 : 8;
   int warps;
-  if (groups > 8) {
-    warps = 8;                                  // one group at a time per warp
+  if (groups > target) {
+    warps = target;                             // one group at a time per warp
   } else {
     const int lanes = wide ? (gs + 3) / 4 : gs;
-    int wpg = 8 / groups;
+    int wpg = target / groups;
     const int useful = (lanes + 31) / 32;
     if (wpg > useful) wpg = useful;
     warps = groups * wpg;

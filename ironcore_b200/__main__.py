@@ -26,8 +26,13 @@ def main(argv=None) -> int:
     p_train.add_argument("--rl", action="store_true", help="run the GRPO loop instead of pre-training")
 
     p_roll = sub.add_parser("rollout", help="sample from a model on the paged KV cache")
-    p_roll.add_argument("--config", required=True)
+    p_roll.add_argument("--config", default=None, help="training YAML; the checkpoint under trainer.model_path is used")
+    p_roll.add_argument("--model", default=None, help="model directory (config.json + model.safetensors) instead of --config")
     p_roll.add_argument("--prompt", default=None)
+    p_roll.add_argument("--prompt-ids", dest="prompt_ids", action="append", default=None,
+                        help="with --model: comma-separated token ids of one prompt; repeat for a batch")
+    p_roll.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="with --model: precision")
+    p_roll.add_argument("--temperature", type=float, default=None, help="with --model (default 0: greedy)")
     p_roll.add_argument("--max-new-tokens", type=int, default=64)
 
     p_exp = sub.add_parser("export", help="write a native checkpoint as a HuggingFace directory")

@@ -3,7 +3,7 @@ rollout engine and write logits (no sampling).
 
 Standard input holds one JSON object per line::
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "q1", "tokens": [12, 4], "want": [1]}, {"id": "q2", "tokens": [9]}], "end": ["q2"]}
 
 The entries of a line form one batch: each continues (or opens) request ``id`` by ``tokens``, and ``want`` indexes the
 tokens to report. Requests under ``end`` are closed once the step has run. Reported logits go to ``DIR/<step>.f32``

@@ -76,12 +76,13 @@ def head_product(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.Ten
     return y.to(x.dtype)
 
 
-def _attend_splits(rows: int, heads: int, max_keys: int) -> int:
-    """Ranges of keys per query row for the tensor-core kernel: about two CTAs per SM, at least four 32-key tiles
-    each."""
+def _attend_splits(rows: int, heads: int, rank: int, max_keys: int) -> int:
+    """Ranges of keys per query row for the tensor-core kernel: as many CTAs as fit on the machine at once (two per
+    SM, three where the rows are narrow), at least four 32-key tiles each."""
     sms = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
-    want = (2 * sms) // max(1, rows * ((heads + 15) // 16))
-    return max(1, min(want, 16, max_keys // 128))
+    groups = (heads + 31) // 32 if heads > 16 else 1
+    slots = sms * (2 if rank > 256 else 3)
+    return max(1, min(slots // max(1, rows * groups), 16, max_keys // 128))
 
 
 def latent_attend(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, block_size: int, seqs: torch.Tensor,
@@ -94,7 +95,7 @@ def latent_attend(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tenso
         out = torch.empty_like(q)
         nsplit, scratch = 1, None
         if q.dtype == torch.bfloat16 and r % 64 == 0 and r <= MMA_MAX_RANK:
-            nsplit = _attend_splits(t, h, max_keys)
+            nsplit = _attend_splits(t, h, r, max_keys)
             if nsplit > 1:
                 scratch = torch.empty(t * h * nsplit * (r + 2), dtype=torch.float32, device=q.device)
         call("icb_latent_attend", ptr(q), ptr(cache), ptr(block_table), ptr(seqs), ptr(positions), ptr(out),

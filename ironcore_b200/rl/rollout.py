@@ -63,7 +63,8 @@ class RolloutEngine:
     @torch.no_grad()
     def step(self, entries: Sequence[Tuple[Hashable, Sequence[int], Optional[Sequence[int]]]]) -> torch.Tensor:
         """``entries``: (request id, its next tokens, places among them whose logits are wanted; None = the last).
-        An unknown id starts a request. Returns logits [wanted, V_local] in entry order."""
+        An unknown id starts a request. Returns logits [wanted, V_local] in entry order, in a buffer that the next
+        step may overwrite."""
         vocab = self.model.vocab_size
         wants, base = [], 0
         for rid, tokens, want in entries:
@@ -80,13 +81,15 @@ class RolloutEngine:
         ids = [e[0] for e in entries]
         if len(set(ids)) != len(ids):
             raise ValueError("a request may appear once in a step")
-        fresh = [i for i in ids if i not in self._requests]
-        for i in fresh:
-            self._requests[i] = self.cache.acquire()
-        seqs = [self._requests[i] for i in ids]
         flat = [t for _, tokens, _ in entries for t in tokens]
         counts = [len(tokens) for _, tokens, _ in entries]
+        fresh = []
         try:
+            for i in ids:
+                if i not in self._requests:
+                    self._requests[i] = self.cache.acquire()
+                    fresh.append(i)
+            seqs = [self._requests[i] for i in ids]
             if not fresh and max(counts) == 1:
                 logits = self._decode(seqs, torch.tensor(flat, dtype=torch.int64))
                 return logits if wants == list(range(len(ids))) else logits[wants]
