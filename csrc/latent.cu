@@ -8,9 +8,10 @@
 //                         latents, writes the latent to its cache row, and the sigmoid of the gates.
 //  * head_product       : out[t, n, :] = B_n a[t, n, :] (optionally times a gate per (t, n)): the query-side and
 //                         output-side products, one small matrix per head, weights streamed once.
-//  * latent_attend_mma  : tensor-core attention of single query rows, 16 or 32 heads per CTA. Latent rows come in tiles
-//                         of 32 tokens by cp.async, double or triple buffered; a tile is both K and V. Four warps own
-//                         a quarter of the rank columns each. The visible range can be cut over CTAs, with
+//  * latent_attend_tc   : attention of single query rows on tcgen05 (rank a multiple of 128 up to 512), see below.
+//  * latent_attend_mma  : the same on mma.sync for the other ranks, 16 or 32 heads per CTA. Latent rows come in tiles
+//                         of 32 tokens by cp.async, double or triple buffered; a tile is both K and V. Every warp owns
+//                         a slice of the rank columns. The visible range can be cut over CTAs, with
 //                         latent_merge joining the parts.
 //  * latent_attend_rows : the same for any rank and type on plain FMAs (fp32 models, ranks beyond 512).
 // A query row is (sequence slot, position): its keys are the `window` tokens that end with itself (window <= 0: all up to itself), so
@@ -133,19 +134,20 @@ __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], uint32_t a0, uint3
 
 constexpr int kHpWarps = 4;
 
-// a: [rows, heads * K], b: [heads, N, K], out: [rows, heads * N]; K a multiple of 32, N of 16. A warp owns 16 output
-// columns of MT * 16 rows. The order of the contraction index inside a group of 32 is free as long as both operands
-// use the same one, so lane (r, c) takes elements [8 c, 8 c + 8) of its rows with one 16-byte load each, which fill
-// the fragments of two consecutive k-steps.
+// a: [rows, heads * K], b: [heads, N, K], out: [rows, heads * N]; K a multiple of 32, N of 16. A CTA makes 16 output
+// columns of MT * 16 rows, its warps taking turns along K and meeting in shared memory: a few rows against many small
+// matrices is bound by latency, so the K loop of a warp is kept short and the grid large. The order of the contraction
+// index inside a group of 32 is free as long as both operands use the same one, so lane (r, c) takes elements
+// [8 c, 8 c + 8) of its rows with one 16-byte load each, which fill the fragments of two consecutive k-steps.
 template <int MT>
 __global__ void __launch_bounds__(kHpWarps * 32)
 head_product_mma_kernel(const uint16_t* __restrict__ a, const uint16_t* __restrict__ b, uint16_t* __restrict__ out,
                         const float* __restrict__ gate, int rows, int heads, int K, int N) {
+  __shared__ float red[kHpWarps][MT * 8][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r = lane >> 2, c = lane & 3;
   const int head = blockIdx.y;
-  const int n0 = (blockIdx.x * kHpWarps + warp) * 16;
-  if (n0 >= N) return;
+  const int n0 = blockIdx.x * 16;
   const int m0 = blockIdx.z * MT * 16;
   const long long lda = (long long)heads * K;
   const uint16_t* b0p = b + ((size_t)head * N + n0 + r) * K + c * 8;
@@ -158,7 +160,7 @@ head_product_mma_kernel(const uint16_t* __restrict__ a, const uint16_t* __restri
     for (int j = 0; j < 2; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll 2
-  for (int k = 0; k < K; k += 32) {
+  for (int k = warp * 32; k < K; k += kHpWarps * 32) {
     const uint4 u0 = *reinterpret_cast<const uint4*>(b0p + k);
     const uint4 u1 = *reinterpret_cast<const uint4*>(b1p + k);
 #pragma unroll
@@ -173,17 +175,26 @@ head_product_mma_kernel(const uint16_t* __restrict__ a, const uint16_t* __restri
     }
   }
 #pragma unroll
-  for (int m = 0; m < MT; ++m) {
+  for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int row = m0 + m * 16 + half * 8 + r;
-      if (row < rows) {
-        const float gt = gate != nullptr ? gate[(size_t)row * heads + head] : 1.f;
-        uint16_t* o = out + ((size_t)row * heads + head) * N + n0 + 2 * c;
+    for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int j = 0; j < 2; ++j)
-          *reinterpret_cast<uint32_t*>(o + 8 * j) = pack_bf16x2(acc[m][j][half * 2] * gt, acc[m][j][half * 2 + 1] * gt);
+      for (int e = 0; e < 4; ++e) red[warp][(m * 2 + j) * 4 + e][lane] = acc[m][j][e];
+  __syncthreads();
+#pragma unroll
+  for (int p = warp; p < MT * 4; p += kHpWarps) {            // p = (m, j, half): a pair of neighbouring columns per lane
+    const int m = p >> 2, j = (p >> 1) & 1, half = p & 1;
+    const int row = m0 + m * 16 + half * 8 + r;
+    if (row < rows) {
+      float lo = 0.f, hi = 0.f;
+#pragma unroll
+      for (int w = 0; w < kHpWarps; ++w) {
+        lo += red[w][(m * 2 + j) * 4 + half * 2][lane];
+        hi += red[w][(m * 2 + j) * 4 + half * 2 + 1][lane];
       }
+      const float gt = gate != nullptr ? gate[(size_t)row * heads + head] : 1.f;
+      *reinterpret_cast<uint32_t*>(out + ((size_t)row * heads + head) * N + n0 + 8 * j + 2 * c) =
+          pack_bf16x2(lo * gt, hi * gt);
     }
   }
 }
@@ -287,8 +298,6 @@ __global__ void __launch_bounds__(kLrChunk) latent_attend_rows_kernel(const Late
 }
 
 // ------------------------------------------------------------------------------------------ latent_attend_mma
-constexpr int kLmThreads = 128;
-constexpr int kLmWarps = kLmThreads / 32;
 constexpr int kLmTok = 32;
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -307,15 +316,23 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 template <int NT, int MT>   // rp = 64 * NT, MT * 16 heads per CTA
 struct LmSmem {
   static constexpr int kRp = 64 * NT;
+  static constexpr int kWarps = 4;
+  static constexpr int kCols = kRp / kWarps;
   static constexpr int kPitch = kRp + 8;                   // rows 16 bytes apart modulo 128: ldmatrix without conflicts
   static constexpr int kStages = NT <= 4 ? 3 : 2;
   static constexpr int tile_bytes = kLmTok * kPitch * 2;
   static constexpr int s_off = kStages * tile_bytes;
   static constexpr int kSPitch = kLmTok + 8;               // float pairs of a fragment row land in distinct banks
-  static constexpr int s_bytes = kLmWarps * MT * 16 * kSPitch * 4;
+  static constexpr int s_bytes = kWarps * MT * 16 * kSPitch * 4;
   static constexpr int p_off = s_off + s_bytes;
   static constexpr int kPPitch = kLmTok + 8;
   static constexpr int p_bytes = MT * 16 * kPPitch * 2;
@@ -323,12 +340,14 @@ struct LmSmem {
   static constexpr int total = row_off + 3 * MT * 16 * 4;
 };
 
-// A warp owns a quarter of the rank columns in both products. Its slice of Q stays in registers; S = Q C^T is the sum
-// of the four slices' parts, which meet in shared memory; O += P C needs nothing from the other warps but P.
+// A warp owns a slice of the rank columns in both products. Its slice of Q stays in registers; S = Q C^T is the sum
+// of the slices' parts, which meet in shared memory; O += P C needs nothing from the other warps but P.
 template <int NT, int MT>
-__global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const LatentAttendArgs a) {
+__global__ void __launch_bounds__(LmSmem<NT, MT>::kWarps * 32, 2) latent_attend_mma_kernel(const LatentAttendArgs a) {
   using L = LmSmem<NT, MT>;
   constexpr int kRows = MT * 16;
+  constexpr int kWarps = L::kWarps, kThreads = kWarps * 32;
+  constexpr int kSteps = L::kCols / 16, kOutTiles = L::kCols / 8;      // k-steps of S, 8-column tiles of O
   extern __shared__ __align__(128) uint8_t lm_smem[];
   const int row = blockIdx.x, h0 = blockIdx.y * kRows, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -349,25 +368,34 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
   const int* bt = a.block_table + (size_t)a.row_seq[row] * a.max_blocks;
   const uint16_t* cache = reinterpret_cast<const uint16_t*>(a.cache);
 
-  auto load_tile = [&](int t) {                              // eight threads per token row, sixteen rows at a time
+  // Eight threads load a token row; a thread's rows (one per kThreads / 8) move on by 32 tokens per tile. Where the
+  // next tile's rows are is looked up one tile ahead, so that the copies never wait for the page table.
+  constexpr int kLoadRows = kLmTok / (kThreads / 8);
+  int next_tok[kLoadRows], next_off[kLoadRows], next_page[kLoadRows], next_blk[kLoadRows];
+#pragma unroll
+  for (int i = 0; i < kLoadRows; ++i) {
+    next_tok[i] = lo + t_begin * kLmTok + (threadIdx.x >> 3) + i * (kThreads / 8);
+    next_page[i] = next_tok[i] / a.block_size;
+    next_off[i] = next_tok[i] - next_page[i] * a.block_size;
+    next_blk[i] = next_tok[i] <= pos ? bt[next_page[i]] : 0;
+  }
+  auto load_tile = [&](int t) {
     if (t < t_end) {
       const uint32_t stage = c_addr + ((t - t_begin) % L::kStages) * L::tile_bytes;
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int tr = (threadIdx.x >> 3) + half * 16;
-        const int tok = lo + t * kLmTok + tr;
-        const bool ok = tok <= pos;
-        const uint16_t* src = cache;
-        if (ok) {
-          const int page = tok / a.block_size;
-          src = cache + ((size_t)bt[page] * a.block_size + (tok - page * a.block_size)) * L::kRp;
-        }
-        const uint32_t dst = stage + tr * (L::kPitch * 2);
+      for (int i = 0; i < kLoadRows; ++i) {
+        const bool ok = next_tok[i] <= pos;
+        const uint16_t* src = ok ? cache + ((size_t)next_blk[i] * a.block_size + next_off[i]) * L::kRp : cache;
+        const uint32_t dst = stage + ((threadIdx.x >> 3) + i * (kThreads / 8)) * (L::kPitch * 2);
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
           const int ch = (threadIdx.x & 7) + j * 8;
           cp_async16(dst + ch * 16, src + ch * 8, ok);
         }
+        next_tok[i] += kLmTok;
+        next_off[i] += kLmTok;
+        while (next_off[i] >= a.block_size) { next_off[i] -= a.block_size; ++next_page[i]; }
+        if (next_tok[i] <= pos) next_blk[i] = bt[next_page[i]];
       }
     }
     cp_async_commit();
@@ -375,14 +403,14 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
 #pragma unroll
   for (int s = 0; s < L::kStages - 1; ++s) load_tile(t_begin + s);
 
-  const int col0 = warp * (16 * NT);                         // this warp's rank columns
-  uint32_t qf[MT][NT][4];
+  const int col0 = warp * L::kCols;                          // this warp's rank columns
+  uint32_t qf[MT][kSteps][4];
   {
     const uint16_t* q = reinterpret_cast<const uint16_t*>(a.q) + (size_t)row * a.heads * L::kRp + col0 + 2 * fc;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-      for (int k = 0; k < NT; ++k)
+      for (int k = 0; k < kSteps; ++k)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int hr = h0 + mt * 16 + fr + (e & 1) * 8;
@@ -390,12 +418,12 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
               ? *reinterpret_cast<const uint32_t*>(q + (size_t)hr * L::kRp + k * 16 + (e >> 1) * 8) : 0u;
         }
   }
-  float acc[MT][2 * NT][4];
+  float acc[MT][kOutTiles][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-    for (int n = 0; n < 2 * NT; ++n) acc[mt][n][0] = acc[mt][n][1] = acc[mt][n][2] = acc[mt][n][3] = 0.f;
-  constexpr int kOwn = kRows / kLmWarps;                     // heads whose softmax this warp does
+    for (int n = 0; n < kOutTiles; ++n) acc[mt][n][0] = acc[mt][n][1] = acc[mt][n][2] = acc[mt][n][3] = 0.f;
+  constexpr int kOwn = kRows / kWarps;                       // heads whose softmax this warp does
   float m[kOwn], l[kOwn];                                    // m: the same in every lane; l: this lane's share
 #pragma unroll
   for (int e = 0; e < kOwn; ++e) { m[e] = -INFINITY; l[e] = 0.f; }
@@ -408,31 +436,29 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
     __syncthreads();                                         // tile t is in place, everybody is done with tile t - 1
     load_tile(t + L::kStages - 1);
     const uint32_t tile = c_addr + ((t - t_begin) % L::kStages) * L::tile_bytes;
-    // ---- this slice's part of the scores, heads x 32 tokens
-    {
-      float sc[MT][4][4];
+    // ---- this slice's part of the scores, heads x 16 tokens at a time
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      float sc[MT][2][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int n = 0; n < 4; ++n) sc[mt][n][0] = sc[mt][n][1] = sc[mt][n][2] = sc[mt][n][3] = 0.f;
+        for (int n = 0; n < 2; ++n) sc[mt][n][0] = sc[mt][n][1] = sc[mt][n][2] = sc[mt][n][3] = 0.f;
 #pragma unroll
-      for (int k = 0; k < NT; ++k) {
+      for (int k = 0; k < kSteps; ++k) {
+        uint32_t b[4];
+        ldsm_x4(b, tile + s_lane + half * 16 * (L::kPitch * 2) + k * 32);
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          uint32_t b[4];
-          ldsm_x4(b, tile + s_lane + half * 16 * (L::kPitch * 2) + k * 32);
-#pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
-            mma_bf16_16816(sc[mt][2 * half], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[0], b[1]);
-            mma_bf16_16816(sc[mt][2 * half + 1], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[2], b[3]);
-          }
+        for (int mt = 0; mt < MT; ++mt) {
+          mma_bf16_16816(sc[mt][0], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[0], b[1]);
+          mma_bf16_16816(sc[mt][1], qf[mt][k][0], qf[mt][k][1], qf[mt][k][2], qf[mt][k][3], b[2], b[3]);
         }
       }
-      float* dst = sS + (warp * kRows + fr) * L::kSPitch + 2 * fc;
+      float* dst = sS + (warp * kRows + fr) * L::kSPitch + half * 16 + 2 * fc;
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
+        for (int n = 0; n < 2; ++n) {
           float* d = dst + mt * 16 * L::kSPitch + n * 8;
           *reinterpret_cast<float2*>(d) = make_float2(sc[mt][n][0], sc[mt][n][1]);
           *reinterpret_cast<float2*>(d + 8 * L::kSPitch) = make_float2(sc[mt][n][2], sc[mt][n][3]);
@@ -447,7 +473,7 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
       for (int e = 0; e < kOwn; ++e) {
         float v = 0.f;
 #pragma unroll
-        for (int w = 0; w < kLmWarps; ++w) v += sS[(w * kRows + warp * kOwn + e) * L::kSPitch + lane];
+        for (int w = 0; w < kWarps; ++w) v += sS[(w * kRows + warp * kOwn + e) * L::kSPitch + lane];
         s[e] = mx[e] = seen ? v * scale_log2 : -INFINITY;
       }
 #pragma unroll
@@ -457,8 +483,8 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
 #pragma unroll
       for (int e = 0; e < kOwn; ++e) {
         const float top = fmaxf(mx[e], m[e]);
-        const float corr = exp2f(m[e] - top);
-        const float p = exp2f(s[e] - top);
+        const float corr = ex2(m[e] - top);
+        const float p = ex2(s[e] - top);
         l[e] = l[e] * corr + p;
         m[e] = top;
         sP[(warp * kOwn + e) * L::kPPitch + lane] = __float2bfloat16(p);
@@ -476,13 +502,13 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
       const float c0 = s_corr[mt * 16 + fr], c1 = s_corr[mt * 16 + fr + 8];
       if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
-        for (int n = 0; n < 2 * NT; ++n) {
+        for (int n = 0; n < kOutTiles; ++n) {
           acc[mt][n][0] *= c0; acc[mt][n][1] *= c0; acc[mt][n][2] *= c1; acc[mt][n][3] *= c1;
         }
       }
     }
 #pragma unroll
-    for (int n = 0; n < 2 * NT; ++n) {
+    for (int n = 0; n < kOutTiles; ++n) {
       uint32_t b[4];
       ldsm_x4_t(b, tile + v_lane + n * 16);
 #pragma unroll
@@ -511,18 +537,322 @@ __global__ void __launch_bounds__(kLmThreads, 2) latent_attend_mma_kernel(const 
           const float inv = s_l[hr] > 0.f ? 1.f / s_l[hr] : 0.f;
           uint16_t* o = reinterpret_cast<uint16_t*>(a.out) + head_row * L::kRp + col;
 #pragma unroll
-          for (int n = 0; n < 2 * NT; ++n)
+          for (int n = 0; n < kOutTiles; ++n)
             *reinterpret_cast<uint32_t*>(o + n * 8) =
                 pack_bf16x2(acc[mt][n][half * 2] * inv, acc[mt][n][half * 2 + 1] * inv);
         } else {
           float* rec = a.part + (head_row * a.nsplit + split) * (L::kRp + 2);
 #pragma unroll
-          for (int n = 0; n < 2 * NT; ++n)
+          for (int n = 0; n < kOutTiles; ++n)
             *reinterpret_cast<float2*>(rec + col + n * 8) = make_float2(acc[mt][n][half * 2], acc[mt][n][half * 2 + 1]);
           if (warp == 0 && fc == 0) *reinterpret_cast<float2*>(rec + L::kRp) = make_float2(s_m[hr], s_l[hr]);
         }
       }
     }
+}
+
+// ------------------------------------------------------------------------------------------- latent_attend_tc
+// tcgen05 form, 16 or 32 heads (HN) of one query row per CTA, one CTA per SM. Heads are far fewer than the 128 rows of
+// an MMA, so both products run transposed, with the cached rows as the M side and the heads as the N side:
+//   S^T [128 tokens, HN]   = C [128 tokens, rank] Q^T              A = C K-major,  B = Q [HN, rank] K-major
+//   O^T [rank, HN]        += C^T [rank, 128 tokens] P^T            A = C MN-major, B = P [HN, tokens] K-major
+// and one copy of a tile of C in shared memory serves both. It arrives through TMA in pairs of 64-column chunks
+// ([128 tokens][64], 128-byte swizzle, sixteen-row boxes so that any page of the cache is a whole number of boxes); a
+// ring of five pairs holds one tile of rank 512 plus the next tile's first pair, and a block of O^T gives its pair back
+// as soon as its MMAs are done. Warp 0 loads, warp 1 issues MMAs, warps 2-5 do the softmax: S^T comes out of TMEM one
+// token per lane, is transposed inside the warp through shared memory to one head per lane, and the four warps exchange
+// only their maxima. The accumulator is rescaled when a head's maximum grows by more than 2^8 (exact: the
+// normalisation uses the same reference), so TMEM is rarely read back. Every wait is bounded.
+constexpr int kLtThreads = 192;
+constexpr int kLtPairs = 5;
+constexpr int kLtTok = 128;
+
+template <int NP, int HN>   // rank = 128 * NP
+struct LtSmem {
+  static constexpr int kRank = 128 * NP;
+  static constexpr int pair_bytes = 2 * kLtTok * 128;
+  static constexpr int q_off = kLtPairs * pair_bytes;
+  static constexpr int q_chunk = HN * 128;
+  static constexpr int p_off = q_off + 2 * NP * q_chunk;
+  static constexpr int t_off = p_off + 2 * q_chunk;
+  static constexpr int kTPitch = 33;
+  static constexpr int x_off = t_off + kLtTok * kTPitch * 4;      // maxima [2][4][32], sums [4][32]
+  static constexpr int bar_off = x_off + 3 * 4 * 32 * 4;
+  static constexpr int total = bar_off + 128 + 1024;              // manual 1 KiB alignment
+  static constexpr int tmem_s = 128;                              // O^T in columns [0, NP * HN), S^T behind
+};
+
+template <int NP, int HN>
+__global__ void __launch_bounds__(kLtThreads, 1)
+latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAttendArgs a, int* status) {
+  using L = LtSmem<NP, HN>;
+  extern __shared__ __align__(1024) uint8_t lt_smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lt_smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* sQ = smem + L::q_off;
+  uint8_t* sP = smem + L::p_off;
+  float* sT = reinterpret_cast<float*>(smem + L::t_off);
+  float* sX = reinterpret_cast<float*>(smem + L::x_off);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::bar_off);
+  uint64_t* full = bars;                 // kLtPairs
+  uint64_t* empty = bars + kLtPairs;     // kLtPairs
+  uint64_t* s_full = bars + 2 * kLtPairs;
+  uint64_t* p_full = s_full + 1;
+  uint64_t* o_full = s_full + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(s_full + 3);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int row = blockIdx.x, h0 = blockIdx.y * HN, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = a.row_pos[row];
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int base = lo & ~15;                                  // tiles start on a sixteen-token box
+  const int tiles = (pos - base) / kLtTok + 1;
+  const int per = (tiles + a.nsplit - 1) / a.nsplit;
+  const int t_begin = split * per, t_end = min(tiles, t_begin + per);
+  const size_t head_row0 = (size_t)row * a.heads + h0;
+  const int heads = min(HN, a.heads - h0);
+
+  if (t_begin >= t_end) {                                     // an empty range (only with several)
+    for (int h = 0; h < heads; ++h) {
+      float* rec = a.part + ((head_row0 + h) * a.nsplit + split) * (L::kRank + 2);
+      for (int i = threadIdx.x; i < L::kRank + 2; i += kLtThreads) rec[i] = i == L::kRank ? -INFINITY : 0.f;
+    }
+    return;
+  }
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kLtPairs; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 1);
+    }
+    mbar_init(s_full, 1);
+    mbar_init(p_full, 128);
+    mbar_init(o_full, 1);
+    *abort_flag = 0;
+    fence_mbar_init();
+    tma_prefetch_desc(&tmC);
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, 256);
+    tmem_relinquish();
+  }
+  {
+    // Q in the K-major swizzled layout: 64-column chunks of [HN rows][128 bytes]
+    const uint16_t* q = reinterpret_cast<const uint16_t*>(a.q) + head_row0 * L::kRank;
+    for (int i = threadIdx.x; i < HN * (L::kRank / 8); i += kLtThreads) {
+      const int hr = i / (L::kRank / 8), piece = i - hr * (L::kRank / 8);
+      const uint4 v = hr < heads ? *reinterpret_cast<const uint4*>(q + (size_t)hr * L::kRank + piece * 8)
+                                 : make_uint4(0u, 0u, 0u, 0u);
+      *reinterpret_cast<uint4*>(sQ + (piece >> 3) * L::q_chunk + hr * 128 + (((piece & 7) ^ (hr & 7)) << 4)) = v;
+    }
+    fence_proxy_async_smem();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_o = *tmem_slot;
+  const uint32_t tmem_s = tmem_o + L::tmem_s;
+  const int n_tiles = t_end - t_begin;
+
+  if (warp == 0) {
+    // ----------------------------- loads: lane = (chunk of the pair, sixteen-token box) -----------------------------
+    const int* bt = a.block_table + (size_t)a.row_seq[row] * a.max_blocks;
+    const int box = lane & 7, chunk = (lane >> 3) & 1;
+    int idx = 0;
+    for (int t = 0; t < n_tiles; ++t) {
+      // boxes past the position repeat its own one: finite values for keys whose weight is zero
+      const int tok = min(base + (t_begin + t) * kLtTok + box * 16, pos & ~15);
+      const int page = tok / a.block_size;
+      const int y = bt[page] * a.block_size + (tok - page * a.block_size);
+      for (int j = 0; j < NP; ++j, ++idx) {
+        const int s = idx % kLtPairs;
+        mbar_wait(&empty[s], ((idx / kLtPairs) & 1) ^ 1, abort_flag, status, kTimeoutSmemEmpty);
+        if (lane == 0) mbar_expect_tx(&full[s], L::pair_bytes);
+        __syncwarp();
+        if (lane < 16)
+          tma_load_2d(smem + s * L::pair_bytes + chunk * (kLtTok * 128) + box * 2048, &tmC, &full[s],
+                      (2 * j + chunk) * 64, y);
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t idesc_s = umma_idesc(128, HN, 1, 0, 0);
+      const uint32_t idesc_o = umma_idesc(128, HN, 1, 1, 0);
+      const uint32_t ring = smem_u32(smem), q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
+      int idx = 0;
+      for (int t = 0; t < n_tiles; ++t) {
+        for (int j = 0; j < NP; ++j) {
+          const int s = (idx + j) % kLtPairs;
+          mbar_wait(&full[s], ((idx + j) / kLtPairs) & 1, abort_flag, status, kTimeoutSmemFull);
+          tc_fence_after();
+          const uint32_t c_addr = ring + s * L::pair_bytes;
+#pragma unroll
+          for (int k = 0; k < 8; ++k)
+            umma_ss(tmem_s, umma_desc_sw128(c_addr + (k >> 2) * (kLtTok * 128) + (k & 3) * 32, 16, 1024),
+                    umma_desc_sw128(q_addr + (2 * j + (k >> 2)) * L::q_chunk + (k & 3) * 32, 16, 1024), idesc_s,
+                    (j > 0 || k > 0) ? 1u : 0u);
+        }
+        umma_commit(s_full);
+        mbar_wait(p_full, t & 1, abort_flag, status, kTimeoutLocalFlag);
+        tc_fence_after();
+        for (int j = 0; j < NP; ++j, ++idx) {
+          const int s = idx % kLtPairs;
+          const uint32_t c_addr = ring + s * L::pair_bytes;
+#pragma unroll
+          for (int k = 0; k < kLtTok / 16; ++k)
+            umma_ss(tmem_o + j * HN, umma_desc_sw128(c_addr + k * 2048, kLtTok * 128, 1024),
+                    umma_desc_sw128(p_addr + (k >> 2) * L::q_chunk + (k & 3) * 32, 16, 1024), idesc_o,
+                    (t > 0 || k > 0) ? 1u : 0u);
+          umma_commit(&empty[s]);
+        }
+      }
+      umma_commit(o_full);
+    }
+    __syncwarp();
+  } else {
+    // ----------------------------------------- softmax and epilogue -----------------------------------------
+    const int q = warp & 3;                                   // TMEM lanes 32 q .. 32 q + 31
+    const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
+    const int head = lane % HN;                               // of this lane after the transposition
+    const int sub = HN == 32 ? 0 : (lane >> 4) * 16;          // its HN tokens of the warp's 32 start here
+    float* my = sT + q * 32 * L::kTPitch;
+    const float scale_log2 = a.scale * 1.4426950408889634f;
+    constexpr int kGroups = (NP * HN + 31) / 32;              // O^T in groups of 32 columns
+    float m_ref = -INFINITY, l = 0.f;
+    for (int t = 0; t < n_tiles; ++t) {
+      mbar_wait(s_full, t & 1, abort_flag, status, kTimeoutTmemFull);
+      tc_fence_after();
+      {
+        uint32_t r[HN];
+        if constexpr (HN == 32) tmem_ld_32x32(tmem_s + lane_off, r);
+        else tmem_ld_32x16(tmem_s + lane_off, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int h = 0; h < HN; ++h) my[lane * L::kTPitch + h] = __uint_as_float(r[h]);
+      }
+      __syncwarp();
+      const int tok0 = base + (t_begin + t) * kLtTok + q * 32 + sub;
+      float v[HN];
+      float mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < HN; ++i) {
+        v[i] = my[(sub + i) * L::kTPitch + head] * scale_log2;
+        if (tok0 + i < lo || tok0 + i > pos) v[i] = -INFINITY;
+        mx = fmaxf(mx, v[i]);
+      }
+      if constexpr (HN == 16) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
+      float* x = sX + (t & 1) * 128;
+      if (sub == 0) x[q * 32 + head] = mx;
+      named_barrier(1, 128);
+      mx = fmaxf(fmaxf(x[head], x[32 + head]), fmaxf(x[64 + head], x[96 + head]));   // the same in all four warps
+      const bool grow = mx > m_ref + 8.f;                     // always in the first tile
+      float factor = 1.f;
+      if (grow) {
+        factor = ex2(m_ref - mx);
+        m_ref = mx;
+        l *= factor;
+      }
+      if (t > 0 && __any_sync(0xffffffffu, grow)) {           // (S^T of this tile is behind O^T of the last: complete)
+#pragma unroll
+        for (int g = 0; g < kGroups; ++g) {
+          uint32_t o[32];
+          tmem_ld_32x32(tmem_o + lane_off + g * 32, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            o[i] = __float_as_uint(__uint_as_float(o[i]) * __shfl_sync(0xffffffffu, factor, i % HN));
+          tmem_st_32x32(tmem_o + lane_off + g * 32, o);
+        }
+        tmem_st_wait();
+      }
+      const int tile_tok = q * 32 + sub;
+      uint8_t* prow = sP + (tile_tok >> 6) * L::q_chunk + head * 128;
+#pragma unroll
+      for (int i = 0; i < HN; i += 8) {
+        float p[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          p[e] = ex2(v[i + e] - m_ref);
+          l += p[e];
+        }
+        uint4 u;
+        u.x = pack_bf16x2(p[0], p[1]); u.y = pack_bf16x2(p[2], p[3]);
+        u.z = pack_bf16x2(p[4], p[5]); u.w = pack_bf16x2(p[6], p[7]);
+        const int piece = ((tile_tok + i) & 63) >> 3;
+        *reinterpret_cast<uint4*>(prow + ((piece ^ (head & 7)) << 4)) = u;
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(p_full);
+    }
+    mbar_wait(o_full, 0, abort_flag, status, kTimeoutTmemFull);
+    tc_fence_after();
+    if constexpr (HN == 16) l += __shfl_xor_sync(0xffffffffu, l, 16);
+    float* sl = sX + 256;
+    if (sub == 0) sl[q * 32 + head] = l;
+    named_barrier(1, 128);
+    l = sl[head] + sl[32 + head] + sl[64 + head] + sl[96 + head];
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+    for (int g = 0; g < kGroups; ++g) {
+      uint32_t o[32];
+      tmem_ld_32x32(tmem_o + lane_off + g * 32, o);
+      tmem_ld_wait();
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const int col = g * 32 + i;
+        const int h = i % HN, rank = (col / HN) * 128 + q * 32 + lane;
+        const float w = __shfl_sync(0xffffffffu, inv, h);
+        if (col < NP * HN && h < heads) {
+          if (a.nsplit == 1)
+            reinterpret_cast<__nv_bfloat16*>(a.out)[(head_row0 + h) * L::kRank + rank] =
+                __float2bfloat16(__uint_as_float(o[i]) * w);
+          else
+            a.part[((head_row0 + h) * a.nsplit + split) * (L::kRank + 2) + rank] = __uint_as_float(o[i]);
+        }
+      }
+    }
+    if (a.nsplit > 1 && q == 0 && sub == 0 && head < heads) {
+      float* rec = a.part + ((head_row0 + head) * a.nsplit + split) * (L::kRank + 2) + L::kRank;
+      rec[0] = m_ref;
+      rec[1] = l;
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_flag) {                                          // let copies in flight land before the memory is given back
+    const long long t0 = clock64();
+    while (clock64() - t0 < 2000000) { __nanosleep(1000); }
+    __syncthreads();
+  }
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_o, 256);
+  }
+}
+
+template <int NP, int HN>
+static int launch_latent_tc_h(const CUtensorMap& tm, const LatentAttendArgs& a, int* status, cudaStream_t st) {
+  auto kern = latent_attend_tc_kernel<NP, HN>;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<NP, HN>::total);
+    if (e != cudaSuccess) return -(int)e;
+    configured = true;
+  }
+  dim3 grid(a.rows, (a.heads + HN - 1) / HN, a.nsplit);
+  kern<<<grid, kLtThreads, LtSmem<NP, HN>::total, st>>>(tm, a, status);
+  return check_launch("latent_attend_tc_kernel");
+}
+template <int NP>
+static int launch_latent_tc(const LatentAttendArgs& a, long long cache_rows, int* status, cudaStream_t st) {
+  CUtensorMap tm;
+  const uint64_t dims[2] = {(uint64_t)a.rp, (uint64_t)cache_rows};
+  const uint64_t strides[1] = {(uint64_t)a.rp * 2};
+  const uint32_t box[2] = {64, 16};
+  const int rc = make_tmap(&tm, kBF16, 2, a.cache, dims, strides, box, true);
+  if (rc) return rc;
+  return a.heads > 16 ? launch_latent_tc_h<NP, 32>(tm, a, status, st) : launch_latent_tc_h<NP, 16>(tm, a, status, st);
 }
 
 // Joins the parts of one (row, head): running maxima are in the log2 domain; an empty part has max -inf and sum 0.
@@ -537,6 +867,7 @@ latent_merge_kernel(const float* __restrict__ part, uint16_t* __restrict__ out, 
   const float inv = l > 0.f ? 1.f / l : 0.f;
   for (int i = threadIdx.x * 2; i < rp; i += 256) {
     float a0 = 0.f, a1 = 0.f;
+#pragma unroll 4
     for (int s = 0; s < nsplit; ++s) {
       const float f = exp2f(rec[(size_t)s * (rp + 2) + rp] - mx);
       const float2 v = *reinterpret_cast<const float2*>(rec + (size_t)s * (rp + 2) + i);
@@ -557,7 +888,7 @@ static int launch_latent_mma_m(const LatentAttendArgs& a, cudaStream_t st) {
     configured = true;
   }
   dim3 grid(a.rows, (a.heads + MT * 16 - 1) / (MT * 16), a.nsplit);
-  kern<<<grid, kLmThreads, LmSmem<NT, MT>::total, st>>>(a);
+  kern<<<grid, LmSmem<NT, MT>::kWarps * 32, LmSmem<NT, MT>::total, st>>>(a);
   return check_launch("latent_attend_mma_kernel");
 }
 template <int NT>
@@ -599,7 +930,7 @@ ICB_API int icb_head_product(const void* a, const void* b, void* out, const floa
     auto A = reinterpret_cast<const uint16_t*>(a);
     auto B = reinterpret_cast<const uint16_t*>(b);
     auto O = reinterpret_cast<uint16_t*>(out);
-    const int gx = (N + 16 * kHpWarps - 1) / (16 * kHpWarps);
+    const int gx = N / 16;
     if (rows <= 16)
       head_product_mma_kernel<1><<<dim3(gx, heads, 1), kHpWarps * 32, 0, st>>>(A, B, O, gate, rows, heads, K, N);
     else if (rows <= 32)
@@ -620,13 +951,15 @@ ICB_API int icb_head_product(const void* a, const void* b, void* out, const floa
 }
 
 // Attention of query rows q [rows, heads, rp] over the latent cache; see the head of this file. bf16 with rp a multiple
-// of 64 up to 512 runs on tensor cores, optionally cut into nsplit ranges with scratch
-// [rows * heads * nsplit * (rp + 2)] floats; everything else on the plain kernel (nsplit is ignored).
+// of 64 up to 512 runs on tensor cores (tcgen05 for multiples of 128, unless `legacy` asks for mma.sync), optionally cut
+// into nsplit ranges with scratch [rows * heads * nsplit * (rp + 2)] floats; everything else on the plain kernel
+// (nsplit is ignored). cache_rows: rows of the cache; block_size a multiple of 16.
 ICB_API int icb_latent_attend(const void* q, const void* cache, const int* block_table, const int* row_seq,
                               const int* row_pos, void* out, float* scratch, int rows, int heads, int rp, int block_size,
-                              int max_blocks, int window, float scale, int nsplit, int dtype, void* stream) {
+                              int max_blocks, int window, float scale, int nsplit, int dtype, void* stream,
+                              long long cache_rows, int* status, int legacy) {
   if (rows <= 0) return 0;
-  if (heads < 1 || rp < 1 || block_size < 1 || max_blocks < 1 || nsplit < 1) return -2;
+  if (heads < 1 || rp < 1 || block_size < 16 || block_size % 16 || max_blocks < 1 || nsplit < 1) return -2;
   if (dtype != kBF16 && dtype != kF32) return -3;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   LatentAttendArgs a;
@@ -636,7 +969,14 @@ ICB_API int icb_latent_attend(const void* q, const void* cache, const int* block
   if (dtype == kBF16 && rp % 64 == 0 && rp <= 512) {
     if (nsplit > 1 && scratch == nullptr) return -4;
     int rc = -2;
-    switch (rp / 64) {
+    if (rp % 128 == 0 && !legacy) {
+      switch (rp / 128) {
+        case 1: rc = launch_latent_tc<1>(a, cache_rows, status, st); break;
+        case 2: rc = launch_latent_tc<2>(a, cache_rows, status, st); break;
+        case 3: rc = launch_latent_tc<3>(a, cache_rows, status, st); break;
+        case 4: rc = launch_latent_tc<4>(a, cache_rows, status, st); break;
+      }
+    } else switch (rp / 64) {
       case 1: rc = launch_latent_mma<1>(a, st); break;
       case 2: rc = launch_latent_mma<2>(a, st); break;
       case 3: rc = launch_latent_mma<3>(a, st); break;

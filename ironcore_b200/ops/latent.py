@@ -16,7 +16,7 @@ from .native import call, dtype_code, ptr, stream_ptr
 P, I, L, F = native.P, native.I, native.L, native.F
 native.register("icb_latent_norm", [P, L, P, P, P, I, P, P, P, P, I, I, I, I, I, F, I, P])
 native.register("icb_head_product", [P, P, P, P, I, I, I, I, I, P])
-native.register("icb_latent_attend", [P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P])
+native.register("icb_latent_attend", [P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, L, P, I])
 
 MMA_MAX_RANK = 512     # widest latent row of the tensor-core attention kernel
 
@@ -76,31 +76,33 @@ def head_product(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.Ten
     return y.to(x.dtype)
 
 
-def _attend_splits(rows: int, heads: int, rank: int, max_keys: int) -> int:
-    """Ranges of keys per query row for the tensor-core kernel: as many CTAs as fit on the machine at once (two per
-    SM, three where the rows are narrow), at least four 32-key tiles each."""
+def _attend_splits(rows: int, heads: int, rank: int, max_keys: int, legacy: bool) -> int:
+    """Ranges of keys per query row for the tensor-core kernels: as many CTAs as the machine holds at once (one per SM
+    for tcgen05; two or three for mma.sync), each with at least two 128-key tiles."""
     sms = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
     groups = (heads + 31) // 32 if heads > 16 else 1
-    slots = sms * (2 if rank > 256 else 3)
-    return max(1, min(slots // max(1, rows * groups), 16, max_keys // 128))
+    slots = sms * ((2 if rank > 256 else 3) if legacy else 1)
+    return max(1, min(slots // max(1, rows * groups), 32, max_keys // (128 if legacy else 256)))
 
 
 def latent_attend(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, block_size: int, seqs: torch.Tensor,
-                  positions: torch.Tensor, *, window: int, scale: float, max_keys: int) -> torch.Tensor:
+                  positions: torch.Tensor, *, window: int, scale: float, max_keys: int,
+                  legacy: bool = False) -> torch.Tensor:
     """q [T, H, R] against latent cache rows [slots, R] -> [T, H, R]: softmax-weighted sum of the latents that row
     (``seqs`` int32, ``positions`` int32) sees. ``window`` <= 0: every earlier token. ``max_keys`` bounds how many
-    keys any row sees."""
+    keys any row sees. ``legacy``: mma.sync where tcgen05 would serve (CUDA, bf16)."""
     t, h, r = q.shape
     if q.is_cuda:
         out = torch.empty_like(q)
         nsplit, scratch = 1, None
         if q.dtype == torch.bfloat16 and r % 64 == 0 and r <= MMA_MAX_RANK:
-            nsplit = _attend_splits(t, h, r, max_keys)
+            legacy = legacy or r % 128 != 0
+            nsplit = _attend_splits(t, h, r, max_keys, legacy)
             if nsplit > 1:
                 scratch = torch.empty(t * h * nsplit * (r + 2), dtype=torch.float32, device=q.device)
         call("icb_latent_attend", ptr(q), ptr(cache), ptr(block_table), ptr(seqs), ptr(positions), ptr(out),
              ptr(scratch), t, h, r, int(block_size), block_table.shape[1], int(window), float(scale), nsplit,
-             dtype_code(q.dtype), stream_ptr())
+             dtype_code(q.dtype), stream_ptr(), cache.shape[0], ptr(native.status_tensor(q.device)), 1 if legacy else 0)
         return out
     out = torch.empty_like(q)
     for i in range(t):

@@ -111,14 +111,15 @@ def test_head_product_kernel(dtype, rows, heads, k, n):
         _close(got, OL.head_product(x, w, gate), dtype)
 
 
-@pytest.mark.parametrize("dtype,rank", [(BF, 64), (BF, 128), (BF, 192), (BF, 320), (BF, 448), (BF, 512), (BF, 576), (F32, 64),
+@pytest.mark.parametrize("dtype,rank", [(BF, 64), (BF, 128), (BF, 192), (BF, 256), (BF, 320), (BF, 384), (BF, 448), (BF, 512), (BF, 576), (F32, 64),
                                         (F32, 192)])
 @pytest.mark.parametrize("heads,window", [(1, 1), (6, 33), (16, 64), (17, 130), (40, 0)])
 def test_latent_attend_kernel(dtype, rank, heads, window):
     """Random keys with one standout per row at the edges of the window, positions around page and tile borders."""
     from ironcore_b200.ops import latent as OL
+    from ironcore_b200.ops import native
 
-    bs, pages, n_seq = 16, 30, 3
+    bs, pages, n_seq = (16, 30, 3) if heads != 17 else (48, 10, 3)
     positions = [0, 1, 15, 16, 31, 32, 33, 63, 64, 127, 130, 299, 470]
     g = torch.Generator().manual_seed(1)
     table = torch.randperm(n_seq * pages, generator=g).to(torch.int32).view(n_seq, pages)
@@ -134,23 +135,25 @@ def test_latent_attend_kernel(dtype, rank, heads, window):
     seqs = torch.tensor([r[0] for r in rows], dtype=torch.int32)
     pos = torch.tensor([r[1] for r in rows], dtype=torch.int32)
     want = OL.latent_attend(q, cache, table, bs, seqs, pos, window=window, scale=0.7, max_keys=471)
-    for keys in (471, 100):                 # cut into ranges, and in one piece
+    for keys, legacy in ((1 << 20, False), (100, False), (1 << 20, True), (100, True)):   # many ranges, and one piece
         got = OL.latent_attend(q.cuda(), cache.cuda(), table.cuda(), bs, seqs.cuda(), pos.cuda(), window=window, scale=0.7,
-                               max_keys=keys)
+                               max_keys=keys, legacy=legacy)
         _close(got, want, dtype)
+    native.check_status()
 
 
 def test_latent_attend_splits_leave_empty_ranges():
     """More ranges than tiles: the empty ones contribute nothing."""
     from ironcore_b200.ops import latent as OL
 
-    cache, q = _rand(64, 64, dtype=BF), _rand(2, 4, 64, seed=1, dtype=BF)
-    table = torch.arange(4, dtype=torch.int32).view(1, 4)
-    seqs, pos = torch.zeros(2, dtype=torch.int32), torch.tensor([0, 40], dtype=torch.int32)
-    want = OL.latent_attend(q, cache, table, 16, seqs, pos, window=0, scale=0.3, max_keys=64)
-    got = OL.latent_attend(q.cuda(), cache.cuda(), table.cuda(), 16, seqs.cuda(), pos.cuda(), window=0, scale=0.3,
-                           max_keys=4096)
-    _close(got, want, BF)
+    for rank in (64, 128):
+        cache, q = _rand(64, rank, dtype=BF), _rand(2, 4, rank, seed=1, dtype=BF)
+        table = torch.arange(4, dtype=torch.int32).view(1, 4)
+        seqs, pos = torch.zeros(2, dtype=torch.int32), torch.tensor([0, 40], dtype=torch.int32)
+        want = OL.latent_attend(q, cache, table, 16, seqs, pos, window=0, scale=0.3, max_keys=64)
+        got = OL.latent_attend(q.cuda(), cache.cuda(), table.cuda(), 16, seqs.cuda(), pos.cuda(), window=0, scale=0.3,
+                               max_keys=4096)
+        _close(got, want, BF)
 
 
 @pytest.mark.parametrize("hd", [64, 128])
