@@ -557,7 +557,8 @@ __global__ void __launch_bounds__(LmSmem<NT, MT>::kWarps * 32, 2) latent_attend_
 //   S^T [128 tokens, HN]   = C [128 tokens, rank] Q^T              A = C K-major,  B = Q [HN, rank] K-major
 //   O^T [rank, HN]        += C^T [rank, 128 tokens] P^T            A = C MN-major, B = P [HN, tokens] K-major
 // and one copy of a tile of C in shared memory serves both. It arrives through TMA in pairs of 64-column chunks
-// ([128 tokens][64], 128-byte swizzle, sixteen-row boxes so that any page of the cache is a whole number of boxes); a
+// ([128 tokens][64], 128-byte swizzle; a box has 16 to 128 rows, the most that page borders allow, and pages of 64 and
+// more tokens keep the number of copies small); a
 // ring of five pairs holds one tile of rank 512 plus the next tile's first pair, and a block of O^T gives its pair back
 // as soon as its MMAs are done. Warp 0 loads, warp 1 issues MMAs, warps 2-5 do the softmax: S^T comes out of TMEM one
 // token per lane, is transposed inside the warp through shared memory to one head per lane, and the four warps exchange
@@ -584,7 +585,7 @@ struct LtSmem {
 
 template <int NP, int HN>
 __global__ void __launch_bounds__(kLtThreads, 1)
-latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAttendArgs a, int* status) {
+latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAttendArgs a, int box_log2, int* status) {
   using L = LtSmem<NP, HN>;
   extern __shared__ __align__(1024) uint8_t lt_smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lt_smem_raw) + 1023) & ~uintptr_t(1023));
@@ -598,14 +599,16 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
   uint64_t* s_full = bars + 2 * kLtPairs;
   uint64_t* p_full = s_full + 1;
   uint64_t* o_full = s_full + 2;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(s_full + 3);
+  uint64_t* q_full = s_full + 3;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(s_full + 4);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int row = blockIdx.x, h0 = blockIdx.y * HN, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = a.row_pos[row];
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  const int base = lo & ~15;                                  // tiles start on a sixteen-token box
+  const int box_rows = 1 << box_log2;
+  const int base = lo & ~(box_rows - 1);                      // tiles start on a box
   const int tiles = (pos - base) / kLtTok + 1;
   const int per = (tiles + a.nsplit - 1) / a.nsplit;
   const int t_begin = split * per, t_end = min(tiles, t_begin + per);
@@ -627,6 +630,7 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
     mbar_init(s_full, 1);
     mbar_init(p_full, 128);
     mbar_init(o_full, 1);
+    mbar_init(q_full, 128);
     *abort_flag = 0;
     fence_mbar_init();
     tma_prefetch_desc(&tmC);
@@ -634,17 +638,6 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
   if (warp == 1) {
     tmem_alloc(tmem_slot, 256);
     tmem_relinquish();
-  }
-  {
-    // Q in the K-major swizzled layout: 64-column chunks of [HN rows][128 bytes]
-    const uint16_t* q = reinterpret_cast<const uint16_t*>(a.q) + head_row0 * L::kRank;
-    for (int i = threadIdx.x; i < HN * (L::kRank / 8); i += kLtThreads) {
-      const int hr = i / (L::kRank / 8), piece = i - hr * (L::kRank / 8);
-      const uint4 v = hr < heads ? *reinterpret_cast<const uint4*>(q + (size_t)hr * L::kRank + piece * 8)
-                                 : make_uint4(0u, 0u, 0u, 0u);
-      *reinterpret_cast<uint4*>(sQ + (piece >> 3) * L::q_chunk + hr * 128 + (((piece & 7) ^ (hr & 7)) << 4)) = v;
-    }
-    fence_proxy_async_smem();
   }
   tc_fence_before();
   __syncthreads();
@@ -654,13 +647,25 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
   const int n_tiles = t_end - t_begin;
 
   if (warp == 0) {
-    // ----------------------------- loads: lane = (chunk of the pair, sixteen-token box) -----------------------------
+    // ----------------------------- loads: lane = (chunk of the pair, box of the tile) -----------------------------
     const int* bt = a.block_table + (size_t)a.row_seq[row] * a.max_blocks;
-    const int box = lane & 7, chunk = (lane >> 3) & 1;
+    const int nb_log2 = 7 - box_log2, nb = 1 << nb_log2;      // boxes per chunk
+    const int box = lane & (nb - 1), chunk = (lane >> nb_log2) & 1;
+    // The ring asks for a tile 256 bytes of a row at a time, which DRAM serves poorly; whole boxes (contiguous rows) are
+    // brought into L2 ahead of it.
+    auto prefetch = [&](int t) {
+      const int tok = base + (t_begin + t) * kLtTok + box * box_rows;
+      if (t < n_tiles && lane < nb && tok <= pos) {
+        const int page = tok / a.block_size;
+        const uint16_t* src = reinterpret_cast<const uint16_t*>(a.cache) +
+                              ((size_t)bt[page] * a.block_size + (tok - page * a.block_size)) * L::kRank;
+        asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(src), "r"(box_rows * L::kRank * 2) : "memory");
+      }
+    };
     int idx = 0;
     for (int t = 0; t < n_tiles; ++t) {
       // boxes past the position repeat its own one: finite values for keys whose weight is zero
-      const int tok = min(base + (t_begin + t) * kLtTok + box * 16, pos & ~15);
+      const int tok = min(base + (t_begin + t) * kLtTok + box * box_rows, pos & ~(box_rows - 1));
       const int page = tok / a.block_size;
       const int y = bt[page] * a.block_size + (tok - page * a.block_size);
       for (int j = 0; j < NP; ++j, ++idx) {
@@ -668,46 +673,58 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
         mbar_wait(&empty[s], ((idx / kLtPairs) & 1) ^ 1, abort_flag, status, kTimeoutSmemEmpty);
         if (lane == 0) mbar_expect_tx(&full[s], L::pair_bytes);
         __syncwarp();
-        if (lane < 16)
-          tma_load_2d(smem + s * L::pair_bytes + chunk * (kLtTok * 128) + box * 2048, &tmC, &full[s],
+        if (lane < 2 * nb)
+          tma_load_2d(smem + s * L::pair_bytes + chunk * (kLtTok * 128) + box * (box_rows * 128), &tmC, &full[s],
                       (2 * j + chunk) * 64, y);
+        if (j == (NP - 1) / 2) prefetch(t + 2);
       }
     }
     __syncwarp();
   } else if (warp == 1) {
-    if (lane == 0) {
-      const uint32_t idesc_s = umma_idesc(128, HN, 1, 0, 0);
-      const uint32_t idesc_o = umma_idesc(128, HN, 1, 1, 0);
-      const uint32_t ring = smem_u32(smem), q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
-      int idx = 0;
-      for (int t = 0; t < n_tiles; ++t) {
-        for (int j = 0; j < NP; ++j) {
-          const int s = (idx + j) % kLtPairs;
-          mbar_wait(&full[s], ((idx + j) / kLtPairs) & 1, abort_flag, status, kTimeoutSmemFull);
-          tc_fence_after();
-          const uint32_t c_addr = ring + s * L::pair_bytes;
+    // The whole warp walks the loops, so that descriptors stay in uniform registers; one lane issues. Descriptors hold
+    // addresses in units of sixteen bytes and shared memory ends below their field, so a step is an addition.
+    const bool leader = elect_one() != 0;
+    const uint32_t idesc_s = umma_idesc(128, HN, 1, 0, 0);
+    const uint32_t idesc_o = umma_idesc(128, HN, 1, 1, 0);
+    const uint64_t c_k = umma_desc_sw128(smem_u32(smem), 16, 1024);                  // C as the K-major operand
+    const uint64_t c_mn = umma_desc_sw128(smem_u32(smem), kLtTok * 128, 1024);       // C as the MN-major operand
+    const uint64_t q_desc = umma_desc_sw128(smem_u32(sQ), 16, 1024);
+    const uint64_t p_desc = umma_desc_sw128(smem_u32(sP), 16, 1024);
+    mbar_wait(q_full, 0, abort_flag, status, kTimeoutLocalFlag);
+    int idx = 0;
+    for (int t = 0; t < n_tiles; ++t) {
+      for (int j = 0; j < NP; ++j) {
+        const int s = (idx + j) % kLtPairs;
+        mbar_wait(&full[s], ((idx + j) / kLtPairs) & 1, abort_flag, status, kTimeoutSmemFull);
+        tc_fence_after();
+        const uint64_t ad = c_k + (uint64_t)(s * (L::pair_bytes >> 4));
+        const uint64_t bd = q_desc + (uint64_t)(j * (2 * L::q_chunk >> 4));
+        if (leader) {
 #pragma unroll
           for (int k = 0; k < 8; ++k)
-            umma_ss(tmem_s, umma_desc_sw128(c_addr + (k >> 2) * (kLtTok * 128) + (k & 3) * 32, 16, 1024),
-                    umma_desc_sw128(q_addr + (2 * j + (k >> 2)) * L::q_chunk + (k & 3) * 32, 16, 1024), idesc_s,
-                    (j > 0 || k > 0) ? 1u : 0u);
+            umma_ss(tmem_s, ad + (((k >> 2) * (kLtTok * 128) + (k & 3) * 32) >> 4),
+                    bd + (((k >> 2) * L::q_chunk + (k & 3) * 32) >> 4), idesc_s, (j > 0 || k > 0) ? 1u : 0u);
         }
-        umma_commit(s_full);
-        mbar_wait(p_full, t & 1, abort_flag, status, kTimeoutLocalFlag);
-        tc_fence_after();
-        for (int j = 0; j < NP; ++j, ++idx) {
-          const int s = idx % kLtPairs;
-          const uint32_t c_addr = ring + s * L::pair_bytes;
+        __syncwarp();
+      }
+      if (leader) umma_commit(s_full);
+      __syncwarp();
+      mbar_wait(p_full, t & 1, abort_flag, status, kTimeoutLocalFlag);
+      tc_fence_after();
+      for (int j = 0; j < NP; ++j, ++idx) {
+        const int s = idx % kLtPairs;
+        const uint64_t ad = c_mn + (uint64_t)(s * (L::pair_bytes >> 4));
+        if (leader) {
 #pragma unroll
           for (int k = 0; k < kLtTok / 16; ++k)
-            umma_ss(tmem_o + j * HN, umma_desc_sw128(c_addr + k * 2048, kLtTok * 128, 1024),
-                    umma_desc_sw128(p_addr + (k >> 2) * L::q_chunk + (k & 3) * 32, 16, 1024), idesc_o,
+            umma_ss(tmem_o + j * HN, ad + (k * 2048 >> 4), p_desc + (((k >> 2) * L::q_chunk + (k & 3) * 32) >> 4), idesc_o,
                     (t > 0 || k > 0) ? 1u : 0u);
           umma_commit(&empty[s]);
         }
+        __syncwarp();
       }
-      umma_commit(o_full);
     }
+    if (leader) umma_commit(o_full);
     __syncwarp();
   } else {
     // ----------------------------------------- softmax and epilogue -----------------------------------------
@@ -718,6 +735,25 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
     float* my = sT + q * 32 * L::kTPitch;
     const float scale_log2 = a.scale * 1.4426950408889634f;
     constexpr int kGroups = (NP * HN + 31) / 32;              // O^T in groups of 32 columns
+    {
+      // Q in the K-major swizzled layout: 64-column chunks of [HN rows][128 bytes]; all loads of a thread in flight
+      const uint16_t* qg = reinterpret_cast<const uint16_t*>(a.q) + head_row0 * L::kRank;
+      constexpr int kPieces = L::kRank / 8, kEach = HN * kPieces / 128;
+      uint4 u[kEach];
+#pragma unroll
+      for (int i = 0; i < kEach; ++i) {
+        const int hr = (i * 128 + (int)threadIdx.x - 64) / kPieces, piece = (i * 128 + (int)threadIdx.x - 64) % kPieces;
+        u[i] = hr < heads ? *reinterpret_cast<const uint4*>(qg + (size_t)hr * L::kRank + piece * 8)
+                          : make_uint4(0u, 0u, 0u, 0u);
+      }
+#pragma unroll
+      for (int i = 0; i < kEach; ++i) {
+        const int hr = (i * 128 + (int)threadIdx.x - 64) / kPieces, piece = (i * 128 + (int)threadIdx.x - 64) % kPieces;
+        *reinterpret_cast<uint4*>(sQ + (piece >> 3) * L::q_chunk + hr * 128 + (((piece & 7) ^ (hr & 7)) << 4)) = u[i];
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(q_full);
+    }
     float m_ref = -INFINITY, l = 0.f;
     for (int t = 0; t < n_tiles; ++t) {
       mbar_wait(s_full, t & 1, abort_flag, status, kTimeoutTmemFull);
@@ -732,13 +768,19 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
       }
       __syncwarp();
       const int tok0 = base + (t_begin + t) * kLtTok + q * 32 + sub;
-      float v[HN];
-      float mx = -INFINITY;
+      float v[HN], mx;
 #pragma unroll
-      for (int i = 0; i < HN; ++i) {
-        v[i] = my[(sub + i) * L::kTPitch + head] * scale_log2;
-        if (tok0 + i < lo || tok0 + i > pos) v[i] = -INFINITY;
-        mx = fmaxf(mx, v[i]);
+      for (int i = 0; i < HN; ++i) v[i] = my[(sub + i) * L::kTPitch + head] * scale_log2;
+      if (base + (t_begin + t) * kLtTok < lo || base + (t_begin + t + 1) * kLtTok > pos + 1) {   // a border tile
+#pragma unroll
+        for (int i = 0; i < HN; ++i)
+          if (tok0 + i < lo || tok0 + i > pos) v[i] = -INFINITY;
+      }
+      {
+        float m4[4] = {v[0], v[1], v[2], v[3]};
+#pragma unroll
+        for (int i = 4; i < HN; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
+        mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
       }
       if constexpr (HN == 16) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
       float* x = sX + (t & 1) * 128;
@@ -767,13 +809,14 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
       }
       const int tile_tok = q * 32 + sub;
       uint8_t* prow = sP + (tile_tok >> 6) * L::q_chunk + head * 128;
+      float l4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int i = 0; i < HN; i += 8) {
         float p[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           p[e] = ex2(v[i + e] - m_ref);
-          l += p[e];
+          l4[e & 3] += p[e];
         }
         uint4 u;
         u.x = pack_bf16x2(p[0], p[1]); u.y = pack_bf16x2(p[2], p[3]);
@@ -784,6 +827,7 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
       fence_proxy_async_smem();
       tc_fence_before();
       mbar_arrive(p_full);
+      l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
     }
     mbar_wait(o_full, 0, abort_flag, status, kTimeoutTmemFull);
     tc_fence_after();
@@ -802,12 +846,13 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
       for (int i = 0; i < 32; ++i) {
         const int col = g * 32 + i;
         const int h = i % HN, rank = (col / HN) * 128 + q * 32 + lane;
-        const float w = __shfl_sync(0xffffffffu, inv, h);
-        if (col < NP * HN && h < heads) {
-          if (a.nsplit == 1)
+        if (a.nsplit == 1) {
+          const float w = __shfl_sync(0xffffffffu, inv, h);
+          if (col < NP * HN && h < heads)
             reinterpret_cast<__nv_bfloat16*>(a.out)[(head_row0 + h) * L::kRank + rank] =
                 __float2bfloat16(__uint_as_float(o[i]) * w);
-          else
+        } else {
+          if (col < NP * HN && h < heads)
             a.part[((head_row0 + h) * a.nsplit + split) * (L::kRank + 2) + rank] = __uint_as_float(o[i]);
         }
       }
@@ -832,7 +877,8 @@ latent_attend_tc_kernel(const __grid_constant__ CUtensorMap tmC, const LatentAtt
 }
 
 template <int NP, int HN>
-static int launch_latent_tc_h(const CUtensorMap& tm, const LatentAttendArgs& a, int* status, cudaStream_t st) {
+static int launch_latent_tc_h(const CUtensorMap& tm, const LatentAttendArgs& a, int box_log2, int* status,
+                              cudaStream_t st) {
   auto kern = latent_attend_tc_kernel<NP, HN>;
   static bool configured = false;
   if (!configured) {
@@ -841,7 +887,7 @@ static int launch_latent_tc_h(const CUtensorMap& tm, const LatentAttendArgs& a, 
     configured = true;
   }
   dim3 grid(a.rows, (a.heads + HN - 1) / HN, a.nsplit);
-  kern<<<grid, kLtThreads, LtSmem<NP, HN>::total, st>>>(tm, a, status);
+  kern<<<grid, kLtThreads, LtSmem<NP, HN>::total, st>>>(tm, a, box_log2, status);
   return check_launch("latent_attend_tc_kernel");
 }
 template <int NP>
@@ -849,32 +895,50 @@ static int launch_latent_tc(const LatentAttendArgs& a, long long cache_rows, int
   CUtensorMap tm;
   const uint64_t dims[2] = {(uint64_t)a.rp, (uint64_t)cache_rows};
   const uint64_t strides[1] = {(uint64_t)a.rp * 2};
-  const uint32_t box[2] = {64, 16};
+  int box_log2 = 4;
+  while (box_log2 < 7 && a.block_size % (2 << box_log2) == 0) ++box_log2;
+  const uint32_t box[2] = {64, 1u << box_log2};
   const int rc = make_tmap(&tm, kBF16, 2, a.cache, dims, strides, box, true);
   if (rc) return rc;
-  return a.heads > 16 ? launch_latent_tc_h<NP, 32>(tm, a, status, st) : launch_latent_tc_h<NP, 16>(tm, a, status, st);
+  return a.heads > 16 ? launch_latent_tc_h<NP, 32>(tm, a, box_log2, status, st)
+                      : launch_latent_tc_h<NP, 16>(tm, a, box_log2, status, st);
 }
 
-// Joins the parts of one (row, head): running maxima are in the log2 domain; an empty part has max -inf and sum 0.
+// Joins the parts of one (row, head): running maxima are in the log2 domain; an empty part has max -inf and sum 0. A
+// thread makes four output values; four parts at a time have all their loads in flight together.
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part, uint16_t* __restrict__ out, int rp, int nsplit) {
   const size_t head_row = blockIdx.x;
   const float* rec = part + head_row * nsplit * (rp + 2);
-  float mx = -INFINITY;
-  for (int s = 0; s < nsplit; ++s) mx = fmaxf(mx, rec[(size_t)s * (rp + 2) + rp]);
-  float l = 0.f;
-  for (int s = 0; s < nsplit; ++s) l += rec[(size_t)s * (rp + 2) + rp + 1] * exp2f(rec[(size_t)s * (rp + 2) + rp] - mx);
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int i = threadIdx.x * 2; i < rp; i += 256) {
-    float a0 = 0.f, a1 = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < nsplit; ++s) {
-      const float f = exp2f(rec[(size_t)s * (rp + 2) + rp] - mx);
-      const float2 v = *reinterpret_cast<const float2*>(rec + (size_t)s * (rp + 2) + i);
-      a0 += f * v.x;
-      a1 += f * v.y;
+  for (int i = threadIdx.x * 4; i < rp; i += 512) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f}, mx = -INFINITY, l = 0.f;
+    for (int s0 = 0; s0 < nsplit; s0 += 4) {
+      float2 ml[4], v0[4], v1[4];
+#pragma unroll
+      for (int s = 0; s < 4; ++s) {
+        const float* r = rec + (size_t)min(s0 + s, nsplit - 1) * (rp + 2);
+        ml[s] = *reinterpret_cast<const float2*>(r + rp);
+        v0[s] = *reinterpret_cast<const float2*>(r + i);
+        v1[s] = *reinterpret_cast<const float2*>(r + i + 2);
+        if (s0 + s >= nsplit) ml[s] = make_float2(-INFINITY, 0.f);
+      }
+      const float top = fmaxf(fmaxf(fmaxf(ml[0].x, ml[1].x), fmaxf(ml[2].x, ml[3].x)), mx);
+      if (top == -INFINITY) continue;
+      const float keep = exp2f(mx - top);
+      mx = top;
+      l *= keep;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[e] *= keep;
+#pragma unroll
+      for (int s = 0; s < 4; ++s) {
+        const float f = exp2f(ml[s].x - top);
+        l += f * ml[s].y;
+        acc[0] += f * v0[s].x; acc[1] += f * v0[s].y; acc[2] += f * v1[s].x; acc[3] += f * v1[s].y;
+      }
     }
-    *reinterpret_cast<uint32_t*>(out + head_row * rp + i) = pack_bf16x2(a0 * inv, a1 * inv);
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    *reinterpret_cast<uint2*>(out + head_row * rp + i) =
+        make_uint2(pack_bf16x2(acc[0] * inv, acc[1] * inv), pack_bf16x2(acc[2] * inv, acc[3] * inv));
   }
 }
 

@@ -17,7 +17,7 @@ import json
 import os
 import sys
 
-BLOCK = 16
+PAGE = 64       # tokens
 
 
 def main(argv=None) -> int:
@@ -49,8 +49,8 @@ def main(argv=None) -> int:
     limit = max(1, args.max_tokens)
     seqs = max(1, min(args.max_seqs, limit))
     # every live request may leave its last page partly filled
-    engine = RolloutEngine(model, config, max_seqs=seqs, max_seq_len=limit, block_size=BLOCK,
-                           num_blocks=(limit + BLOCK - 1) // BLOCK + seqs)
+    engine = RolloutEngine(model, config, max_seqs=seqs, max_seq_len=limit, block_size=PAGE,
+                           num_blocks=(limit + PAGE - 1) // PAGE + seqs)
     if mesh.is_rank_zero():
         os.makedirs(args.out, exist_ok=True)
     for line in sys.stdin:

@@ -29,9 +29,11 @@ class TransformerProgram:
     and scatter the rotated K / V rows into cache pages; all other rows append and attend over their pages. Tensor
     parallelism uses the plain (non sequence-parallel) layout, one all-reduce after each row-parallel projection."""
 
-    def __init__(self, model, config, max_seqs: int, max_seq_len: int, block_size: int, num_blocks: Optional[int]):
+    def __init__(self, model, config, max_seqs: int, max_seq_len: int, block_size: Optional[int],
+                 num_blocks: Optional[int]):
         self.model, self.config = model, config
         m = config.model
+        block_size = block_size or config.rl.kv_block_size
         self.tp_group = mesh.get_tensor_model_parallel_group()
         self.tp = mesh.get_tensor_model_parallel_world_size()
         self.tp_rank = mesh.get_tensor_model_parallel_rank()
@@ -154,13 +156,17 @@ class TransformerProgram:
 
 
 class StreamProgram:
-    """Residual-stream models: latent rows and shift states in a :class:`LatentCache`, fp32 logits."""
+    """Residual-stream models: latent rows and shift states in a :class:`LatentCache`, fp32 logits. Pages hold 64 tokens
+    unless asked otherwise: a latent row is narrow, and the decode kernel copies a page with one box per 64 columns."""
 
-    def __init__(self, model, config, max_seqs: int, max_seq_len: int, block_size: int, num_blocks: Optional[int]):
+    PAGE = 64
+
+    def __init__(self, model, config, max_seqs: int, max_seq_len: int, block_size: Optional[int],
+                 num_blocks: Optional[int]):
         self.model = model
         table = model.embedding.word_embeddings.weight
-        self.cache = model.model.make_cache(max_seqs, max_seq_len, block_size, num_blocks, device=table.device,
-                                            dtype=table.dtype)
+        self.cache = model.model.make_cache(max_seqs, max_seq_len, block_size or self.PAGE, num_blocks,
+                                            device=table.device, dtype=table.dtype)
 
     def refresh(self):
         self.model.model.refresh()

@@ -46,7 +46,7 @@ class RolloutEngine:
         self.tp_rank = mesh.get_tensor_model_parallel_rank()
         self.device = next(model.parameters()).device
         self.program = make_program(model, config, max_seqs=max_seqs, max_seq_len=max_seq_len,
-                                    block_size=block_size or config.rl.kv_block_size, num_blocks=num_blocks)
+                                    block_size=block_size, num_blocks=num_blocks)
         self.cache = self.program.cache
         self.max_seqs = max_seqs
         on_gpu = self.device.type == "cuda"

@@ -119,7 +119,7 @@ def test_latent_attend_kernel(dtype, rank, heads, window):
     from ironcore_b200.ops import latent as OL
     from ironcore_b200.ops import native
 
-    bs, pages, n_seq = (16, 30, 3) if heads != 17 else (48, 10, 3)
+    bs, pages, n_seq = {17: (48, 10, 3), 16: (64, 8, 3), 40: (128, 4, 3)}.get(heads, (16, 30, 3))
     positions = [0, 1, 15, 16, 31, 32, 33, 63, 64, 127, 130, 299, 470]
     g = torch.Generator().manual_seed(1)
     table = torch.randperm(n_seq * pages, generator=g).to(torch.int32).view(n_seq, pages)
