@@ -132,71 +132,88 @@ __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], uint32_t a0, uint3
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-constexpr int kHpWarps = 4;
-
-// a: [rows, heads * K], b: [heads, N, K], out: [rows, heads * N]; K a multiple of 32, N of 16. A CTA makes 16 output
-// columns of MT * 16 rows, its warps taking turns along K and meeting in shared memory: a few rows against many small
+// a: [rows, heads * K], b: [heads, N, K], out: [rows, heads * N]; K a multiple of 32, N of 16. A CTA makes 32 output
+// columns of MT * 16 rows, its W warps taking turns along K and meeting in shared memory: a few rows against many small
 // matrices is bound by latency, so the K loop of a warp is kept short and the grid large. The order of the contraction
 // index inside a group of 32 is free as long as both operands use the same one, so lane (r, c) takes elements
 // [8 c, 8 c + 8) of its rows with one 16-byte load each, which fill the fragments of two consecutive k-steps.
-template <int MT>
-__global__ void __launch_bounds__(kHpWarps * 32)
+template <int MT, int W>
+__global__ void __launch_bounds__(W * 32)
 head_product_mma_kernel(const uint16_t* __restrict__ a, const uint16_t* __restrict__ b, uint16_t* __restrict__ out,
                         const float* __restrict__ gate, int rows, int heads, int K, int N) {
-  __shared__ float red[kHpWarps][MT * 8][32];
+  constexpr int kVals = MT * 16;                             // accumulators of a lane: MT x 4 column tiles x 4
+  __shared__ float red[4][kVals][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r = lane >> 2, c = lane & 3;
   const int head = blockIdx.y;
-  const int n0 = blockIdx.x * 16;
+  const int n0 = blockIdx.x * 32;
   const int m0 = blockIdx.z * MT * 16;
+  const bool wide = n0 + 16 < N;                             // (N is a multiple of 16: the last CTA may have half)
   const long long lda = (long long)heads * K;
-  const uint16_t* b0p = b + ((size_t)head * N + n0 + r) * K + c * 8;
-  const uint16_t* b1p = b0p + (size_t)8 * K;
+  const uint16_t* bp = b + ((size_t)head * N + n0 + r) * K + c * 8;
   const uint16_t* ap = a + (size_t)head * K + c * 8;
-  float acc[MT][2][4];
+  float acc[MT][4][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int j = 0; j < 2; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
+    for (int j = 0; j < 4; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll 2
-  for (int k = warp * 32; k < K; k += kHpWarps * 32) {
-    const uint4 u0 = *reinterpret_cast<const uint4*>(b0p + k);
-    const uint4 u1 = *reinterpret_cast<const uint4*>(b1p + k);
+  for (int k = warp * 32; k < K; k += W * 32) {
+    uint4 u[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      u[j] = (j < 2 || wide) ? *reinterpret_cast<const uint4*>(bp + (size_t)j * 8 * K + k) : zero;
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
       const int ra = m0 + m * 16 + r;
       const uint4 v0 = ra < rows ? *reinterpret_cast<const uint4*>(ap + (size_t)ra * lda + k) : zero;
       const uint4 v1 = ra + 8 < rows ? *reinterpret_cast<const uint4*>(ap + (size_t)(ra + 8) * lda + k) : zero;
-      mma_bf16_16816(acc[m][0], v0.x, v1.x, v0.y, v1.y, u0.x, u0.y);
-      mma_bf16_16816(acc[m][0], v0.z, v1.z, v0.w, v1.w, u0.z, u0.w);
-      mma_bf16_16816(acc[m][1], v0.x, v1.x, v0.y, v1.y, u1.x, u1.y);
-      mma_bf16_16816(acc[m][1], v0.z, v1.z, v0.w, v1.w, u1.z, u1.w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        mma_bf16_16816(acc[m][j], v0.x, v1.x, v0.y, v1.y, u[j].x, u[j].y);
+        mma_bf16_16816(acc[m][j], v0.z, v1.z, v0.w, v1.w, u[j].z, u[j].w);
+      }
     }
   }
+  auto put = [&](int w) {
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+    for (int i = 0; i < kVals; ++i) red[w][i][lane] = acc[i >> 4][(i >> 2) & 3][i & 3];
+  };
+  if constexpr (W == 8) {
+    if (warp >= 4) put(warp - 4);
+    __syncthreads();
+    if (warp < 4) {
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) red[warp][(m * 2 + j) * 4 + e][lane] = acc[m][j][e];
+      for (int i = 0; i < kVals; ++i) acc[i >> 4][(i >> 2) & 3][i & 3] += red[warp][i][lane];
+    }
+    __syncthreads();
+  }
+  if (warp < 4) put(warp);
   __syncthreads();
 #pragma unroll
-  for (int p = warp; p < MT * 4; p += kHpWarps) {            // p = (m, j, half): a pair of neighbouring columns per lane
-    const int m = p >> 2, j = (p >> 1) & 1, half = p & 1;
+  for (int p = warp; p < MT * 8; p += W) {                   // p = (m, j, half): a pair of neighbouring columns per lane
+    const int m = p >> 3, j = (p >> 1) & 3, half = p & 1;
     const int row = m0 + m * 16 + half * 8 + r;
-    if (row < rows) {
+    if (row < rows && (j < 2 || wide)) {
       float lo = 0.f, hi = 0.f;
 #pragma unroll
-      for (int w = 0; w < kHpWarps; ++w) {
-        lo += red[w][(m * 2 + j) * 4 + half * 2][lane];
-        hi += red[w][(m * 2 + j) * 4 + half * 2 + 1][lane];
+      for (int w = 0; w < 4; ++w) {
+        lo += red[w][m * 16 + j * 4 + half * 2][lane];
+        hi += red[w][m * 16 + j * 4 + half * 2 + 1][lane];
       }
       const float gt = gate != nullptr ? gate[(size_t)row * heads + head] : 1.f;
       *reinterpret_cast<uint32_t*>(out + ((size_t)row * heads + head) * N + n0 + 8 * j + 2 * c) =
           pack_bf16x2(lo * gt, hi * gt);
     }
   }
+}
+
+template <int MT>
+static void launch_head_product(const uint16_t* a, const uint16_t* b, uint16_t* out, const float* gate, int rows,
+                                int heads, int K, int N, cudaStream_t st) {
+  const dim3 grid((N + 31) / 32, heads, (rows + MT * 16 - 1) / (MT * 16));
+  if (K >= 256) head_product_mma_kernel<MT, 8><<<grid, 256, 0, st>>>(a, b, out, gate, rows, heads, K, N);
+  else head_product_mma_kernel<MT, 4><<<grid, 128, 0, st>>>(a, b, out, gate, rows, heads, K, N);
 }
 
 // The same product in fp32: one CTA per (row, head), a warp per output value.
@@ -994,16 +1011,10 @@ ICB_API int icb_head_product(const void* a, const void* b, void* out, const floa
     auto A = reinterpret_cast<const uint16_t*>(a);
     auto B = reinterpret_cast<const uint16_t*>(b);
     auto O = reinterpret_cast<uint16_t*>(out);
-    const int gx = N / 16;
-    if (rows <= 16)
-      head_product_mma_kernel<1><<<dim3(gx, heads, 1), kHpWarps * 32, 0, st>>>(A, B, O, gate, rows, heads, K, N);
-    else if (rows <= 32)
-      head_product_mma_kernel<2><<<dim3(gx, heads, 1), kHpWarps * 32, 0, st>>>(A, B, O, gate, rows, heads, K, N);
-    else {
-      const int gz = (rows + 63) / 64;
-      if (gz > 65535) return -2;
-      head_product_mma_kernel<4><<<dim3(gx, heads, gz), kHpWarps * 32, 0, st>>>(A, B, O, gate, rows, heads, K, N);
-    }
+    if (rows > 64 * 65535) return -2;
+    if (rows <= 16) launch_head_product<1>(A, B, O, gate, rows, heads, K, N, st);
+    else if (rows <= 32) launch_head_product<2>(A, B, O, gate, rows, heads, K, N, st);
+    else launch_head_product<4>(A, B, O, gate, rows, heads, K, N, st);
   } else if (dtype == kF32) {
     head_product_f32_kernel<<<dim3(rows, heads), 128, 0, st>>>(reinterpret_cast<const float*>(a),
                                                                reinterpret_cast<const float*>(b),

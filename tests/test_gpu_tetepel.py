@@ -101,7 +101,8 @@ def test_latent_norm_kernel(dtype, rows, q_rank, rank, heads):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("rows,heads,k,n", [(1, 3, 64, 64), (17, 2, 128, 192), (33, 5, 64, 512), (150, 4, 512, 128)])
+@pytest.mark.parametrize("rows,heads,k,n", [(1, 3, 64, 64), (17, 2, 128, 192), (33, 5, 64, 512), (150, 4, 512, 128),
+                                            (9, 2, 576, 80), (70, 3, 96, 16)])
 def test_head_product_kernel(dtype, rows, heads, k, n):
     from ironcore_b200.ops import latent as OL
 
