@@ -27,7 +27,13 @@ def project(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dty
     if use_native(x):
         return kernels.mm_nt(x, weight, out_dtype=out_dtype)
     if x.dtype == torch.float32:
-        return x @ weight.t()
+        if not (x.is_cuda and torch.backends.cuda.matmul.allow_tf32):
+            return x @ weight.t()
+        torch.backends.cuda.matmul.allow_tf32 = False      # a 32-bit model is 32-bit, whatever training switched on
+        try:
+            return x @ weight.t()
+        finally:
+            torch.backends.cuda.matmul.allow_tf32 = True
     return (x.float() @ weight.float().t()).to(out_dtype)
 
 

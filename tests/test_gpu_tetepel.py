@@ -214,6 +214,20 @@ def test_model_on_the_engine(case, precision):
         assert T.error(got, want) < LIMIT[precision], (cuts, T.error(got, want))
 
 
+def test_fp32_models_ignore_the_tf32_switch():
+    cfg = CASES["aligned"]
+    w, toks = T.weights(cfg), T.tokens(cfg, 20)
+    model, c = T.build(cfg, w, "float32", device="cuda")
+    before = torch.backends.cuda.matmul.allow_tf32
+    try:
+        torch.backends.cuda.matmul.allow_tf32 = True
+        got = T.feed(T.engine(model, c), cfg, toks, [15, 1])
+        assert torch.backends.cuda.matmul.allow_tf32
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = before
+    assert T.error(got, T.reference(cfg, w, toks)) < LIMIT["float32"]
+
+
 def test_bf16_error_is_rounding():
     """On a model without sharp scores the bf16 path stays within a few per cent at every position."""
     cfg = T.config([T.layer(heads=4, dim=64, vdim=64, q_rank=48, kv_rank=64, window=40, scale=0.125, ff=96)] * 2, width=128,
