@@ -233,13 +233,14 @@ def bench_stream_kernels(size: str, report) -> None:
         x, m, g = rand(b, h, k), rand(h, n_out, k), (torch.rand(b, h, device=dev) if gated else None)
         return lambda: latent.head_product(x, m, g)
 
-    def gemm():
-        x, m = rand(b, d), rand(h * hd, d)
+    def gemm(k, n_out):
+        x, m = rand(b, k), rand(n_out, k)
         return lambda: kernels.mm_nt(x, m)
 
     emit("head_product, query side", lambda: product(hd, r, False), nbytes=2 * h * (r * hd + b * (hd + r)), seqs=b)
     emit("head_product, output side", lambda: product(r, hd, True), nbytes=2 * h * (r * hd + b * (hd + r)), seqs=b)
-    emit("decode gemm (llama, o proj)", gemm, nbytes=2 * (h * hd * d + b * (d + h * hd)), seqs=b)
+    for label, k, n_out in (("o proj", d, h * hd), ("as many weights as a head product", r, h * hd)):
+        emit(f"decode gemm (llama, {label})", lambda: gemm(k, n_out), nbytes=2 * (n_out * k + b * (k + n_out)), seqs=b)
 
 
 def run(args) -> int:
@@ -255,7 +256,7 @@ def run(args) -> int:
     for size in ([args.size] if args.size else list(SIZES)):
         bench_stream_kernels(size, report)
         if not args.kernels_only:
-            bench_models(size, max(args.steps, 32), args.warmup, report)
+            bench_models(size, max(args.steps, 128), args.warmup, report)
     report({"workload": "serving", "data": "synthetic", "dtype": "bf16", "clocks": sampler.stop(),
             "l2": "kernel inputs rotate over copies that exceed it twice; model weights exceed it"})
     return 0
