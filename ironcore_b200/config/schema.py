@@ -162,7 +162,7 @@ class MoEConfig(BaseConfig):
 
 @dataclass
 class ModelConfig(BaseConfig):
-    name: Optional[str] = opt(None, "model family name (gpt2, llama, gemma1, qwen, phi1, phi2, dummy, ...)")
+    name: Optional[str] = opt(None, "model family name (gpt2, llama, gemma1, qwen, phi1, phi2, tetepel, dummy, ...)")
     d_model: int = opt(512, "hidden size")
     d_ffn: int = opt(2048, "feed-forward hidden size")
     num_layers: int = opt(2, "number of transformer layers")
