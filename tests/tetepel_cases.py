@@ -29,6 +29,8 @@ def cases():
                           width=96, groups=12, streams=4, vocab=128, loop={"start": 0, "stop": 1, "times": 1}),
         "wide_heads": config([layer(heads=18, dim=100, vdim=72, q_rank=24, kv_rank=130, window=9, scale=0.1)], width=56,
                              groups=2, streams=3),
+        "beyond_the_fast_kernels": config([layer(heads=2, dim=140, vdim=40, q_rank=200, kv_rank=530, window=11, scale=0.08)],
+                                          width=64, groups=2, streams=2),
     }
 
 
