@@ -1,5 +1,5 @@
 // Flash attention forward for sm_100a: causal / full, GQA, optional document
-// boundaries (cu_seqlens), sliding window, per-head output gate, head_dim 64 or 128, bf16 or fp16.
+// boundaries (cu_seqlens), sliding window or chunks, per-head output gate, head_dim 64 or 128, bf16 or fp16.
 //
 // One CTA owns 128 query rows of one head. Warp 0 streams K and V tiles (128 rows)
 // with TMA into 2-stage rings, warp 1 issues tcgen05.mma for S = Q K^T (TMEM,
@@ -18,6 +18,7 @@
 // Every wait is bounded; on timeout the status word is set and the CTA drains.
 #include "host_common.h"
 #include "ptx.cuh"
+#include "visible.cuh"
 
 namespace icb {
 
@@ -26,7 +27,7 @@ constexpr int kFaThreads = 192;
 struct FlashFwdArgs {
   int batch, seq_len, hq, hkv;        // seq_len: tokens per sequence (max when cu_seqlens is used)
   const int* cu_seqlens;              // [batch + 1] or null (then sequence b spans [b*seq_len, (b+1)*seq_len))
-  void* out;                          // [T, hq, HD]
+  void* out;                          // [T, out_stride], heads HD apart
   float* lse;                         // [hq, T] natural-log sum-exp
   long long total_tokens;
   float scale_log2;                   // softmax scale * log2(e)
@@ -36,8 +37,9 @@ struct FlashFwdArgs {
   const unsigned long long* drop_seed;  // device word; read when drop_thr > 0
   int drop_thr;                       // keep a probability when its hash byte >= drop_thr (0: no dropout)
   float drop_scale;                   // 256 / (256 - drop_thr)
-  int window;                         // causal only: query i sees keys j with i - j < window (0: no limit)
+  Visible see;                        // causal only: window / chunk in front of the query
   const float* gate;                  // [T, hq] factor of a head's output row, or null
+  long long out_stride;               // elements between output rows
 };
 
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -117,8 +119,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   const int q0 = qt * 128;
   const int n_kv_total = (seq_len + BN - 1) / BN;
   const int kv_end = args.causal ? min((q0 + 128 + BN - 1) / BN, n_kv_total) : n_kv_total;
-  // key tiles that end before the window of the tile's first query row are not visited
-  const int kv_first = args.window > 0 ? max(0, q0 - args.window + 1) / BN : 0;
+  // key tiles that end before what the tile's first query row sees are not visited
+  const int kv_first = first_visible(args.see, q0) / BN;
+  const int lo_last = first_visible(args.see, q0 + 127);              // the last row sees the least of the past
   const int n_kv = kv_end - kv_first;
 
   if (threadIdx.x == 0) {
@@ -228,6 +231,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const int row = q * 32 + lane;
     const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
     const int q_idx = q0 + row;  // position inside the sequence
+    const int kv_lo = first_visible(args.see, q_idx);
     float m_ref = -INFINITY;     // reference max (log2 domain, scaled)
     float l_sum = 0.f;
     const bool dropout = args.drop_thr > 0;
@@ -246,9 +250,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tc_fence_before();
       mbar_arrive(&s_empty[s]);
       const int kv0 = (kv_first + j) * BN;
-      const int kv_lo = args.window > 0 ? q_idx - args.window : -1;      // last key that this row no longer sees
       const bool need_mask = (args.causal && kv0 + BN > q0) || (kv0 + BN > seq_len) ||
-                             (args.window > 0 && kv0 <= q0 + 127 - args.window);
+                             kv0 < lo_last;
       float m_tile = -INFINITY;
 #pragma unroll
       for (int c = 0; c < NC; ++c) {
@@ -257,7 +260,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           float x = __uint_as_float(r[c][i]) * args.scale_log2;
           if (need_mask) {
             const int kv_idx = kv0 + c * 32 + i;
-            if (kv_idx >= seq_len || (args.causal && kv_idx > q_idx) || kv_idx <= kv_lo) x = -INFINITY;
+            if (kv_idx >= seq_len || (args.causal && kv_idx > q_idx) || kv_idx < kv_lo) x = -INFINITY;
           }
           r[c][i] = __float_as_uint(x);
           m_tile = fmaxf(m_tile, x);
@@ -342,7 +345,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const long long tok = (long long)seq_start + q_idx;
       float inv_l = l_sum > 0.f ? 1.0f / l_sum : 0.f;
       if (args.gate != nullptr && valid) inv_l *= args.gate[(size_t)tok * args.hq + head];
-      uint8_t* orow = reinterpret_cast<uint8_t*>(args.out) + ((size_t)tok * args.hq + head) * HD * 2;
+      uint8_t* orow = reinterpret_cast<uint8_t*>(args.out) + ((size_t)tok * args.out_stride + (size_t)head * HD) * 2;
 #pragma unroll
       for (int c = 0; c < HD / 32; ++c) {
         uint32_t o[32];
@@ -423,16 +426,19 @@ using namespace icb;
 // [batch + 1]) gives document boundaries in the flat token stream; seq_len is then the maximum length.
 // dropout_p > 0 drops attention probabilities with probability round(256 p) / 256 under the mask that the
 // device word *dropout_seed selects (the backward pass must be given the same word).
-// window > 0 (causal only): a query's keys are the `window` tokens that end with itself. gate (optional, fp32 [T, hq]) multiplies a
-// head's output row.
+// window > 0 (causal only): a query's keys are the `window` tokens that end with itself; chunk > 0 (causal only): those of its own
+// chunk of that many tokens, counted from the sequence's start. gate (optional, fp32 [T, hq]) multiplies a head's output row.
+// out_stride: elements between output rows (0: hq * hd), a multiple of 8.
 ICB_API int icb_flash_fwd(const void* q, const void* k, const void* v, void* out, float* lse, int batch, int seq_len,
                           long long total_tokens, int hq, int hkv, int hd, long long q_stride, long long kv_stride,
                           const int* cu_seqlens, int causal, float scale, int dtype, int* status, void* stream_,
                           float dropout_p, const unsigned long long* dropout_seed, int wide, int window,
-                          const float* gate) {
+                          const float* gate, int chunk, long long out_stride) {
   if (hd != 64 && hd != 128) return -2;
   if (hq % hkv != 0) return -3;
-  if (window > 0 && !causal) return -5;
+  if ((window > 0 || chunk > 0) && !causal) return -5;
+  if (out_stride == 0) out_stride = (long long)hq * hd;
+  if (out_stride % 8) return -6;
   if (batch <= 0 || seq_len <= 0) return 0;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   CUtensorMap tmQ, tmK, tmV;
@@ -455,8 +461,9 @@ ICB_API int icb_flash_fwd(const void* q, const void* k, const void* v, void* out
   if (a.drop_thr > 0 && dropout_seed == nullptr) return -4;
   a.drop_seed = dropout_seed;
   a.drop_scale = 256.0f / (256 - a.drop_thr);
-  a.window = window > 0 ? window : 0;
+  a.see = Visible{window > 0 ? window : 0, chunk > 0 ? chunk : 0};
   a.gate = gate;
+  a.out_stride = out_stride;
   dim3 grid((seq_len + 127) / 128, hq, batch);
   if (bn == 64) {
     if (hd == 64) return launch_flash_fwd<64, 64>(tmQ, tmK, tmV, a, grid, stream);

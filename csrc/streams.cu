@@ -8,7 +8,8 @@
 //   hs   = h + (h_prev - h) * shift                 blend with the previous token's h (optional)
 // which is one pass here: the streams are read once and written once per sublayer, everything in fp32.
 // The first boundary takes x_s = table[token] * scale instead of the write step; the last one has in = 1 and no
-// streams to write, and visits only the rows somebody asked for (row_map).
+// streams to write, and visits only the rows somebody asked for (row_map). Where a pass of a looped block starts, every
+// stream also gets a vector of that pass (add) and, if asked for, the embedding row once more.
 //
 // The previous token's h of a row is, in this order: the carried value of the row handled just before by the same
 // CTA; recomputed from the old streams when that row belongs to another CTA (this is why the streams are written to
@@ -25,10 +26,11 @@ constexpr int kMaxStreams = 16;
 constexpr int kStreamMaxWarps = 16;
 
 struct StreamArgs {
-  const long long* tokens;      // first boundary: token ids [T]
-  const void* table;            // embedding rows (pitch ld_table) or null
+  const long long* tokens;      // token ids [T] for the embedding rows
+  const void* table;            // embedding rows (pitch ld_table) or null; with x_in they are added to the streams
   long long ld_table, table_rows;   // ids outside the table give zeros
   float table_scale;
+  const float* add;             // [D], added to every stream, or null
   const float* x_in;            // [rows, S, D] old streams (null at the first boundary)
   float* x_out;                 // [T, S, D] new streams or null
   const void* y;                // finished sublayer's result, pitch ldy
@@ -121,7 +123,7 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
       if (first && a.row_pos[r] > 0) before = a.prev + (size_t)seq * D;
     }
     const T* table_row = nullptr;
-    if (!write_step) {
+    if (a.table != nullptr) {
       const long long id = a.tokens[src];
       if (id >= 0 && id < a.table_rows) table_row = reinterpret_cast<const T*>(a.table) + id * a.ld_table;
     }
@@ -137,6 +139,20 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
         float u[V];
 #pragma unroll
         for (int v = 0; v < V; ++v) u[v] = 0.f;
+        float e[V];                                     // what every stream gets besides the write step
+#pragma unroll
+        for (int v = 0; v < V; ++v) e[v] = 0.f;
+        if (table_row != nullptr) {
+          load_vec<T, V>(table_row + col, e);
+#pragma unroll
+          for (int v = 0; v < V; ++v) e[v] *= a.table_scale;
+        }
+        if (a.add != nullptr) {
+          float p[V];
+          load_vec<float, V>(a.add + col, p);
+#pragma unroll
+          for (int v = 0; v < V; ++v) e[v] += p[v];
+        }
         if (write_step) {
           float x[SMAX][V], yv[V];
 #pragma unroll
@@ -155,7 +171,7 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
             if (t < S) {
               float n[V];
 #pragma unroll
-              for (int v = 0; v < V; ++v) n[v] = s_out[t] * yv[v];
+              for (int v = 0; v < V; ++v) n[v] = fmaf(s_out[t], yv[v], e[v]);
 #pragma unroll
               for (int s = 0; s < SMAX; ++s)
                 if (s < S) {
@@ -168,12 +184,6 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
             }
           }
         } else {
-          float e[V];
-#pragma unroll
-          for (int v = 0; v < V; ++v) e[v] = 0.f;
-          if (table_row != nullptr) load_vec<T, V>(table_row + col, e);
-#pragma unroll
-          for (int v = 0; v < V; ++v) e[v] *= a.table_scale;
           for (int t = 0; t < S; ++t) {
             if (xo_row != nullptr) store_vec<float, V>(xo_row + (size_t)t * D + col, e);
 #pragma unroll
@@ -260,10 +270,11 @@ static int launch_stream(const StreamArgs& a, bool wide, int blocks, int threads
 using namespace icb;
 
 // One sublayer boundary of the residual streams (see the head of this file). dtype is that of table, y, r, h and hs:
-// bf16 or fp32; everything else is fp32. x_in == null selects the first boundary (tokens, table). x_out must not
-// alias x_in. row_map and a shift exclude each other. rows_per_block <= 0 lets the launcher choose.
+// bf16 or fp32; everything else is fp32. x_in == null selects the first boundary (tokens, table); with x_in, a table adds
+// its rows to the streams, as add [D] (optional) does. x_out must not alias x_in. row_map and a shift exclude each
+// other. rows_per_block <= 0 lets the launcher choose.
 ICB_API int icb_stream_boundary(const long long* tokens, const void* table, long long ld_table, long long table_rows,
-                                float table_scale,
+                                float table_scale, const float* add,
                                 const float* x_in, float* x_out, const void* y, long long ldy, const void* r,
                                 long long ldr, const float* rb, const float* mix, const float* out, const int* row_map,
                                 const float* in, const float* norm_w, int groups, float eps, void* h, void* hs,
@@ -274,10 +285,11 @@ ICB_API int icb_stream_boundary(const long long* tokens, const void* table, long
   if (dtype != kBF16 && dtype != kF32) return -3;
   if (x_in == nullptr ? (tokens == nullptr || table == nullptr) : (y == nullptr || x_in == x_out)) return -4;
   if (r != nullptr && rb == nullptr) return -4;
+  if (table != nullptr && tokens == nullptr) return -4;
   if (hs != nullptr && (row_map != nullptr || shift == nullptr || row_seq == nullptr || row_pos == nullptr || prev == nullptr))
     return -5;
   StreamArgs a;
-  a.tokens = tokens; a.table = table; a.ld_table = ld_table; a.table_rows = table_rows; a.table_scale = table_scale;
+  a.tokens = tokens; a.table = table; a.ld_table = ld_table; a.table_rows = table_rows; a.table_scale = table_scale; a.add = add;
   a.x_in = x_in; a.x_out = x_out; a.y = y; a.ldy = ldy; a.r = r; a.ldr = ldr; a.rb = rb; a.mix = mix; a.out = out;
   a.row_map = row_map; a.in = in; a.norm_w = norm_w; a.groups = groups; a.eps = eps;
   a.h = h; a.hs = hs; a.ldh = ldh; a.shift = shift; a.prev = prev; a.state = state;

@@ -8,13 +8,13 @@ from __future__ import annotations
 
 import json
 from pathlib import Path
-from typing import Callable, Dict, Tuple
+from typing import Callable, Dict, Optional, Tuple
 
 import torch
 
 from ..config.loader import validate_config
 from ..config.schema import MainConfig
-from ..layers.latent_attention import Stored, stored
+from ..layers.mixer import Stored, stored
 from .hf_interop import read_hf_state_dict
 
 
@@ -27,23 +27,54 @@ def _need(doc: dict, *path):
     return node
 
 
-# --------------------------------------------------------------------------- Tetepel
-def tetepel_config(doc: dict, precision: str = "bfloat16") -> MainConfig:
+Shapes = Optional[Dict[str, Tuple[int, ...]]]       # tensor name -> shape, where sizes are not in the document
+
+
+def _stream_config(doc: dict, precision: str, **model) -> MainConfig:
+    """What the documents of the residual-stream families have in common."""
     layers = _need(doc, "layers")
-    first = layers[0] if layers else {}
-    heads = int((first.get("mixer") or {}).get("heads", 1))
     c = MainConfig()
-    c.model(name="tetepel", d_model=int(_need(doc, "width")), vocab_size=int(_need(doc, "vocab")),
-            num_layers=len(layers), layer_specs=list(layers), layer_loop=doc.get("loop") or None,
-            residual_streams=int(_need(doc, "streams")), norm_groups=int(_need(doc, "norm", "groups")),
-            ln_eps=float(_need(doc, "norm", "eps")), embed_scale=float(_need(doc, "embedding", "scale")),
-            num_attention_heads=heads, num_attention_groups=heads, head_dim=int((first.get("mixer") or {}).get("dim", 1)),
-            d_ffn=int((first.get("mlp") or {}).get("ff", 0)), activation_type="geglu", precision=precision,
-            untie_embed=False, dropout_embd=0.0, dropout_attn=0.0, dropout_mlp=0.0, reset_position_ids=False,
-            reset_attention_mask=False)
+    c.model(d_model=int(_need(doc, "width")), vocab_size=int(_need(doc, "vocab")), num_layers=len(layers),
+            layer_loop=doc.get("loop") or None, ln_eps=float(_need(doc, "norm", "eps")),
+            embed_scale=float(_need(doc, "embedding", "scale")), precision=precision, dropout_embd=0.0, dropout_attn=0.0,
+            dropout_mlp=0.0, reset_position_ids=False, reset_attention_mask=False, **model)
     c.data(task_type="synthetic", vocab_size=int(doc["vocab"]))
     c.trainer(micro_batch_size=1, train_batch_size=1, gradient_accumulation_steps=None)
     return validate_config(c)
+
+
+def _stream_tensors(model) -> Dict[str, Stored]:
+    """Tensor name of the checkpoint -> where the model keeps it."""
+    d, v = model.model.d_model, model.vocab_size
+    out = {"embed": stored(model.embedding.word_embeddings.weight.data[:v, :d]),
+           "final.norm": stored(model.output_layernorm.weight.data)}
+    if model.untied:
+        out["head"] = stored(model.output_layer.weight.data[:d, :v].t())
+    out.update(model.model.stored_tensors())
+    return out
+
+
+def _first_sizes(layers, attention: str = "") -> dict:
+    """Head counts and sizes of the first layer that has them (informational: layers have sizes of their own)."""
+    for spec in layers:
+        m = spec.get("mixer") or {}
+        m = m.get(attention, {}) if attention else m
+        if "heads" in m:
+            return dict(num_attention_heads=int(m["heads"]), num_attention_groups=int(m.get("kv_heads", m["heads"])),
+                        head_dim=int(m["dim"]))
+    return dict(num_attention_heads=1, num_attention_groups=1, head_dim=1)
+
+
+def _first_ff(layers) -> int:
+    return next((int(s["mlp"]["ff"]) for s in layers if s.get("mlp")), 0)
+
+
+# --------------------------------------------------------------------------- Tetepel
+def tetepel_config(doc: dict, precision: str = "bfloat16", shapes: Shapes = None) -> MainConfig:
+    layers = _need(doc, "layers")
+    return _stream_config(doc, precision, name="tetepel", layer_specs=list(layers), activation_type="geglu",
+                          residual_streams=int(_need(doc, "streams")), norm_groups=int(_need(doc, "norm", "groups")),
+                          d_ffn=_first_ff(layers), untie_embed=False, **_first_sizes(layers))
 
 
 def tetepel_document(config) -> dict:
@@ -53,17 +84,45 @@ def tetepel_document(config) -> dict:
             "streams": m.residual_streams, "vocab": m.vocab_size, "width": m.d_model}
 
 
-def tetepel_tensors(model) -> Dict[str, Stored]:
-    """Tensor name of the checkpoint -> where the model keeps it."""
-    out = {"embed": stored(model.embedding.word_embeddings.weight.data[:model.vocab_size, :model.model.d_model]),
-           "final.norm": stored(model.output_layernorm.weight.data)}
-    for i, layer in enumerate(model.model.layers):
-        out.update({f"l{i}.{name}": v for name, v in layer.stored_tensors().items()})
-    return out
+# --------------------------------------------------------------------------- Kedavik
+_KEDAVIK_RANKS = {"decay_rank": "a1", "gate_rank": "g1"}      # sizes that only the tensors of the right branch tell
 
 
+def kedavik_config(doc: dict, precision: str = "bfloat16", shapes: Shapes = None) -> MainConfig:
+    layers = []
+    for i, spec in enumerate(_need(doc, "layers")):
+        spec = dict(spec)
+        if spec.get("type") == "parallel":
+            right = dict(_need(spec, "mixer", "right"))
+            for key, tensor in _KEDAVIK_RANKS.items():
+                shape = (shapes or {}).get(f"l{i}.mix.right.{tensor}")
+                if shape is not None:
+                    right[key] = int(shape[0])
+            spec["mixer"] = {**spec["mixer"], "right": right}
+        layers.append(spec)
+    return _stream_config(doc, precision, name="kedavik", layer_specs=layers, activation_type="gelu", d_ffn=_first_ff(layers),
+                          residual_mult=float(_need(doc, "residual_mult")), untie_embed=True, lm_head_bias=False,
+                          **_first_sizes(layers, "left"))
+
+
+def kedavik_document(config) -> dict:
+    m = config.model
+    layers = []
+    for spec in m.layer_specs:
+        if spec.get("type") == "parallel":
+            right = {k: v for k, v in spec["mixer"]["right"].items() if k not in _KEDAVIK_RANKS}
+            spec = {**spec, "mixer": {**spec["mixer"], "right": right}}
+        layers.append(spec)
+    return {"architecture": "Kedavik", "embedding": {"scale": 1.0 if m.embed_scale is None else m.embed_scale},
+            "layers": layers, "loop": m.layer_loop, "norm": {"eps": m.ln_eps}, "residual_mult": m.residual_mult,
+            "vocab": m.vocab_size, "width": m.d_model}
+
+
+# "architecture" of config.json -> (configuration from document, precision and tensor shapes; document from
+# configuration; places of the checkpoint's tensors in the model)
 ARCHITECTURES: Dict[str, Tuple[Callable, Callable, Callable]] = {
-    "Tetepel": (tetepel_config, tetepel_document, tetepel_tensors),
+    "Tetepel": (tetepel_config, tetepel_document, _stream_tensors),
+    "Kedavik": (kedavik_config, kedavik_document, _stream_tensors),
 }
 
 
@@ -92,7 +151,7 @@ def load_tensors(model, tensors: Dict[str, torch.Tensor]) -> None:
         t = tensors[name]
         if tuple(t.shape) != place.shape:
             raise ValueError(f"{name}: expected shape {place.shape}, got {tuple(t.shape)}")
-        place.view.copy_(t.reshape(place.view.shape))
+        place.put(t)
     for p in model.parameters():      # the views above go through .data: tell whoever derives values from weights
         torch._C._autograd._unsafe_set_version_counter((p,), (p._version + 1,))
     model.model.refresh()
@@ -110,9 +169,10 @@ def load_pretrained(path, precision: str = "bfloat16", device=None):
     from ..models import LanguageModel
 
     doc = read_document(path)
-    config = ARCHITECTURES[doc["architecture"]][0](doc, precision)
+    weights = read_hf_state_dict(path)
+    config = ARCHITECTURES[doc["architecture"]][0](doc, precision, {k: tuple(t.shape) for k, t in weights.items()})
     model = LanguageModel(config, device=device).eval()
-    load_tensors(model, read_hf_state_dict(path))
+    load_tensors(model, weights)
     return model, config
 
 
@@ -127,6 +187,6 @@ def save_pretrained(model, config, path) -> Path:
     out.mkdir(parents=True, exist_ok=True)
     (out / "config.json").write_text(json.dumps(document(config), indent=1, sort_keys=True))
     dtype = next(model.parameters()).dtype
-    save_file({k: v.view.reshape(v.shape).to("cpu", dtype).contiguous() for k, v in tensors(model).items()},
+    save_file({k: v.value().to("cpu", dtype).contiguous() for k, v in tensors(model).items()},
               str(out / "model.safetensors"))
     return out

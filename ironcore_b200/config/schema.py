@@ -162,7 +162,7 @@ class MoEConfig(BaseConfig):
 
 @dataclass
 class ModelConfig(BaseConfig):
-    name: Optional[str] = opt(None, "model family name (gpt2, llama, gemma1, qwen, phi1, phi2, tetepel, dummy, ...)")
+    name: Optional[str] = opt(None, "model family name (gpt2, llama, gemma1, qwen, phi1, phi2, tetepel, kedavik, dummy, ...)")
     d_model: int = opt(512, "hidden size")
     d_ffn: int = opt(2048, "feed-forward hidden size")
     num_layers: int = opt(2, "number of transformer layers")
@@ -206,6 +206,17 @@ class ModelConfig(BaseConfig):
     layer_loop: Optional[dict] = opt(None, "residual-stream families: {start, stop, times}, the block "
                                      "[start, stop) is evaluated `times` times, sharing its weights")
     residual_streams: int = opt(1, "residual streams per token (hyper-connections)")
+    stream_mixing: Optional[bool] = opt(None, "residual-stream families: learned weights of reading, writing and mixing the "
+                                        "streams around every sublayer (None = family default)")
+    residual_gates: Optional[bool] = opt(None, "residual-stream families: an element-wise gate on every sublayer's result "
+                                         "(None = family default)")
+    token_shift: Optional[bool] = opt(None, "residual-stream families: blend a mixer's input with the previous token's "
+                                      "(None = family default)")
+    residual_mult: float = opt(1.0, "residual-stream families without learned stream weights: factor of every sublayer's "
+                               "result")
+    loop_inputs: Optional[bool] = opt(None, "residual-stream families: before every pass of the looped block add a learned "
+                                      "vector of that pass, and before every pass but the first the embedding output "
+                                      "(None = family default)")
     norm_groups: int = opt(1, "residual-stream families: equal parts of a row that are normed on their own")
     hf_model_type: Optional[str] = opt(None, "HuggingFace model_type")
     hf_architecture: Optional[str] = opt(None, "HuggingFace architecture name")

@@ -14,28 +14,14 @@ matrix pitches to 16 bytes. The padding is zero and changes no result. ``stored_
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, NamedTuple, Optional, Tuple
+from typing import Dict, List
 
 import torch
 import torch.nn as nn
 
 from ..ops import latent as OL
 from ..ops.functional import use_native
-
-
-def pad_to(n: int, unit: int) -> int:
-    return (n + unit - 1) // unit * unit
-
-
-class Stored(NamedTuple):
-    """A checkpoint tensor inside a (padded, packed) parameter: a view of its values and its stored shape."""
-
-    view: torch.Tensor
-    shape: Tuple[int, ...]
-
-
-def stored(view: torch.Tensor, *shape: int) -> Stored:
-    return Stored(view, tuple(shape) or tuple(view.shape))
+from .mixer import CacheSpec, PackedLinear, Stored, pad_to, stored
 
 
 @dataclass
@@ -54,17 +40,6 @@ class LatentAttentionSpec:
         return LatentAttentionSpec(heads=int(mixer["heads"]), dim=int(mixer["dim"]), vdim=int(mixer["vdim"]),
                                    q_rank=int(mixer["q_rank"]), kv_rank=int(mixer["kv_rank"]),
                                    scale=float(mixer["scale"]), window=int(mask.get("size") or 0))
-
-
-class PackedLinear(nn.Module):
-    """A weight in checkpoint orientation [out, in] whose rows and columns may be padded or hold several matrices."""
-
-    def __init__(self, rows: int, cols: int, dtype=None, device=None):
-        super().__init__()
-        self.weight = nn.Parameter(torch.zeros((rows, cols), dtype=dtype, device=device))
-
-    def forward(self, x: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-        return OL.project(x, self.weight, out_dtype)
 
 
 class LatentAttention(nn.Module):
@@ -105,6 +80,13 @@ class LatentAttention(nn.Module):
             "o": stored(self.out.weight.data.view(-1, s.heads, self.vd)[:d, :, :s.vdim], d, s.heads * s.vdim),
         }
 
+    def native_symbols(self) -> List[str]:
+        fast = self.out.weight.dtype in (torch.bfloat16, torch.float16)
+        return ["icb_latent_norm"] + (["icb_flash_fwd"] if fast and self.flash else [])
+
+    def cache_spec(self) -> CacheSpec:
+        return CacheSpec(rows={"latent": self.c_width}, window=self.spec.window)
+
     def refresh(self) -> torch.Tensor:
         """[heads, c_width, qd]: the key expansion transposed for the query side, rebuilt in place (captured graphs
         keep its address) when ``kv_up`` has changed."""
@@ -126,7 +108,7 @@ class LatentAttention(nn.Module):
         whole = batch.kind == "prompt" and self.flash and (use_native(h) or not h.is_cuda)
         z = self.in_proj(h, torch.float32)
         cq, c, gate = OL.latent_norm(z, self.q_layernorm, self.c_layernorm, s.heads, self.eps, q_width=self.q_width,
-                                     c_width=self.c_width, dtype=h.dtype, cache=cache.latent[run], slots=batch.slots,
+                                     c_width=self.c_width, dtype=h.dtype, cache=cache.rows[run]["latent"], slots=batch.slots,
                                      want_latent=whole)
         q = self.q_up(cq)
         if whole:
@@ -135,7 +117,7 @@ class LatentAttention(nn.Module):
         else:
             q = OL.head_product(q.view(-1, s.heads, self.qd), self.refresh())
             keys = min(s.window, batch.max_context) if s.window > 0 else batch.max_context
-            o = OL.latent_attend(q, cache.latent[run], cache.block_table, cache.block_size, batch.seqs,
+            o = OL.latent_attend(q, cache.rows[run]["latent"], cache.block_table, cache.block_size, batch.seqs,
                                  batch.positions, window=s.window, scale=s.scale, max_keys=keys)
             v_up = self.kv_up.weight.data[s.heads * self.qd:].view(s.heads, self.vd, -1)
             ctx = OL.head_product(o, v_up, gate).reshape(h.shape[0], -1)

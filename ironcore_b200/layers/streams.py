@@ -12,23 +12,31 @@ import torch.nn as nn
 
 from ..ops.latent import project
 from .activations import Activation
-from .latent_attention import PackedLinear, Stored, pad_to, stored
+from .mixer import PackedLinear, Stored, pad_to, stored
 from .norm import GroupedRMSNorm
 
 
 class StreamPort(nn.Module):
     """How one sublayer reads from and writes to the streams: ``u = sum_s read[s] x_s``, then (all from the old
-    values) ``x_t <- sum_s mix[s, t] x_s + write[t] y``; and the grouped norm of what it reads."""
+    values) ``x_t <- sum_s mix[s, t] x_s + write[t] y``; and the grouped norm of what it reads. The stream weights are
+    parameters, or without ``learned`` constants: plain residual streams whose results count ``gain`` times."""
 
-    def __init__(self, d_model: int, streams: int, groups: int, eps: float, device=None):
+    def __init__(self, d_model: int, streams: int, groups: int, eps: float, device=None, learned: bool = True,
+                 gain: float = 1.0):
         super().__init__()
+        self.learned = learned
         kw = dict(dtype=torch.float32, device=device)
-        self.read = nn.Parameter(torch.full((streams,), 1.0 / streams, **kw))
-        self.write = nn.Parameter(torch.ones(streams, **kw))
-        self.mix = nn.Parameter(torch.eye(streams, **kw))
+        for name, value in (("read", torch.full((streams,), 1.0 / streams, **kw)),
+                            ("write", torch.full((streams,), float(gain), **kw)), ("mix", torch.eye(streams, **kw))):
+            if learned:
+                self.register_parameter(name, nn.Parameter(value))
+            else:
+                self.register_buffer(name, value, persistent=False)
         self.norm = GroupedRMSNorm(d_model, groups, eps, device=device)
 
     def reset(self):
+        if not self.learned:
+            return
         with torch.no_grad():
             self.read.fill_(1.0 / self.read.numel())
             self.write.fill_(1.0)
@@ -50,6 +58,27 @@ class ResidualGate(nn.Module):
 
     def stored_tensors(self) -> Dict[str, Stored]:
         return {"": stored(self.proj.weight.data[:self.d_model, :self.d_model]), ".b": stored(self.bias.data)}
+
+
+class DenseMLP(nn.Module):
+    """down(act(up h + b)) + b, for residual streams without gates."""
+
+    def __init__(self, d_model: int, d_ffn: int, activation: str = "gelu", dtype=None, device=None):
+        super().__init__()
+        self.d_model, self.d_ffn = d_model, d_ffn
+        width, f_width = pad_to(d_model, 8), pad_to(d_ffn, 8)
+        self.activation = Activation(activation)
+        self.up_proj = PackedLinear(f_width, width, dtype=dtype, device=device, bias=True)
+        self.down_proj = PackedLinear(width, f_width, dtype=dtype, device=device, bias=True)
+
+    def forward(self, h: torch.Tensor):
+        """h [T, width] -> (result [T, width], no gate)."""
+        return self.down_proj(self.activation(self.up_proj(h))), None
+
+    def stored_tensors(self) -> Dict[str, Stored]:
+        d, f = self.d_model, self.d_ffn
+        return {"mlp.up": stored(self.up_proj.weight.data[:f, :d]), "mlp.up.b": stored(self.up_proj.bias.data[:f]),
+                "mlp.down": stored(self.down_proj.weight.data[:d, :f]), "mlp.down.b": stored(self.down_proj.bias.data[:d])}
 
 
 class GatedStreamMLP(nn.Module):

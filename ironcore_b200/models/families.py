@@ -9,15 +9,17 @@ from __future__ import annotations
 
 import math
 
-FAMILIES = ("GPT", "LLAMA", "GEMMA1", "GEMMA", "QWEN", "PHI1", "PHI2", "MISTRAL", "MOE", "DUMMY", "TETEPEL")
-STREAM_FAMILIES = ("TETEPEL",)      # several residual streams, layers listed in model.layer_specs
+FAMILIES = ("GPT", "LLAMA", "GEMMA1", "GEMMA", "QWEN", "PHI1", "PHI2", "MISTRAL", "MOE", "DUMMY", "TETEPEL",
+            "KEDAVIK")
+STREAM_FAMILIES = ("TETEPEL", "KEDAVIK")      # fp32 residual streams, layers listed in model.layer_specs
 
 
 def family_of(name: str) -> str:
     if not name:
         raise ValueError("model.name is required (e.g. gpt2-small, llama, gemma1, qwen, phi2, dummy)")
     up = name.upper().replace("-", "").replace("_", "")
-    for fam in ("GEMMA1", "GEMMA", "PHI1", "PHI2", "LLAMA", "QWEN", "MISTRAL", "GPT", "MOE", "DUMMY", "TETEPEL"):
+    for fam in ("GEMMA1", "GEMMA", "PHI1", "PHI2", "LLAMA", "QWEN", "MISTRAL", "GPT", "MOE", "DUMMY", "TETEPEL",
+                "KEDAVIK"):
         if up.startswith(fam):
             return "GEMMA1" if fam == "GEMMA" else fam
     raise ValueError(f"model '{name}' is not a supported family ({', '.join(FAMILIES)})")
@@ -30,6 +32,12 @@ def resolve_family_defaults(model_cfg) -> str:
     pe = m.positional_embedding
     if fam in STREAM_FAMILIES:
         pe.type, m.ln_type, m.no_bias = "none", "rmsnorm", True
+        learned = fam == "TETEPEL"
+        m.activation_type = "geglu" if learned else "gelu"
+        for switch, default in (("stream_mixing", learned), ("residual_gates", learned), ("token_shift", learned),
+                                ("loop_inputs", fam == "KEDAVIK")):
+            if getattr(m, switch) is None:
+                setattr(m, switch, default)
         if m.layer_specs:
             m.num_layers = len(m.layer_specs)
     if m.qkv_bias is None:

@@ -115,8 +115,9 @@ class LanguageModel(BaseModule):
             self.output_layernorm = get_norm(config, dtype, device)
         self.untied = bool(m.untie_embed)
         if self.untied:
-            self.output_layer = ColumnParallelLinear(m.d_model, self.padded_vocab_size, bias=bool(m.lm_head_bias),
-                                                     dtype=dtype, device=device)
+            rows = self.model.width if self.family in STREAM_FAMILIES else m.d_model
+            self.output_layer = ColumnParallelLinear(rows, self.padded_vocab_size, bias=bool(m.lm_head_bias), dtype=dtype,
+                                                     device=device)
         self.reset_position_ids = m.reset_position_ids
         self.reset_attention_mask = m.reset_attention_mask
         self.eod_mask_loss = m.eod_mask_loss
@@ -138,6 +139,8 @@ class LanguageModel(BaseModule):
             self.model.init_special()
             with torch.no_grad():
                 self.embedding.word_embeddings.weight[:, self.model.d_model:].zero_()
+                if self.untied:
+                    self.output_layer.weight[self.model.d_model:].zero_()
         tp_rank = mesh.get_tensor_model_parallel_rank()
         # zero the padded vocabulary rows / columns
         with torch.no_grad():
@@ -219,14 +222,20 @@ class LanguageModel(BaseModule):
         h = self.step_hidden(batch, cache)
         if h.shape[0] == 0:
             return torch.empty((0, self.padded_vocab_size), dtype=torch.float32, device=h.device)
+        if self.untied:
+            return project(h, self.output_layer.weight, torch.float32, transposed=True)
         return project(h, self.embedding.word_embeddings.weight, torch.float32)
 
     def native_symbols(self):
         """Entry points of the kernel library that serving this model calls (see ``ops.native.require``)."""
-        names = ["icb_stream_boundary", "icb_latent_norm"]
-        if self.dtype in (torch.bfloat16, torch.float16):
-            names += ["icb_gemm", "icb_gemm_2sm", "icb_glu_fwd", "icb_flash_fwd"]
-        return names if self.family in STREAM_FAMILIES else []
+        if self.family not in STREAM_FAMILIES:
+            return []
+        names = ["icb_stream_boundary"]
+        for layer in self.model.layers:
+            names += layer.mixer.native_symbols()
+        if self.embedding.word_embeddings.weight.dtype in (torch.bfloat16, torch.float16):
+            names += ["icb_gemm", "icb_gemm_2sm", "icb_glu_fwd"]
+        return sorted(set(names))
 
     def _stream_hidden(self, input_ids: torch.Tensor) -> torch.Tensor:
         """[B, S] ids -> final-normed rows [B * S, width], with a cache that lives for this call only."""

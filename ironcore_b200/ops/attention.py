@@ -13,7 +13,7 @@ from .native import call, dtype_code, ptr, stream_ptr
 native.register("icb_flash_fwd", [native.P] * 5 + [native.I, native.I, native.L, native.I, native.I, native.I,
                                                    native.L, native.L, native.P, native.I, native.F, native.I,
                                                    native.P, native.P, native.F, native.P, native.I, native.I,
-                                                   native.P])
+                                                   native.P, native.I, native.L])
 native.register("icb_flash_bwd", [native.P] * 11 + [native.I, native.I, native.L, native.I, native.I, native.I,
                                                     native.L, native.L, native.L, native.L, native.P, native.I,
                                                     native.F, native.I, native.P, native.P, native.F, native.P])
@@ -102,25 +102,37 @@ def flash_fwd(qkv: torch.Tensor, hq: int, hkv: int, hd: int, seq_len: int, *, cu
     call("icb_flash_fwd", base, base + hq * hd * es, base + (hq + hkv) * hd * es, ptr(out), ptr(lse), batch, s, t,
          hq, hkv, hd, stride, stride, ptr(cu_seqlens), 1 if causal else 0, float(scale if scale else hd ** -0.5),
          dtype_code(qkv.dtype), ptr(native.status_tensor(qkv.device)), stream_ptr(), float(dropout_p),
-         ptr(dropout_seed), 1 if wide_tiles else 0, 0, None)
+         ptr(dropout_seed), 1 if wide_tiles else 0, 0, None, 0, 0)
     return out, lse
+
+
+def flash_fwd_heads(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, hq: int, hkv: int, hd: int,
+                    cu_seqlens: torch.Tensor, max_seqlen: int, *, scale: float, window: int = 0, chunk: int = 0,
+                    gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention of ``q`` [T, hq * hd], ``k`` and ``v`` [T, hkv * hd] (column slices of any row pitch, k and v of
+    the same) within the documents of ``cu_seqlens`` (int32 [n + 1], the longest being ``max_seqlen``). ``window`` > 0:
+    query i sees keys j with ``i - j < window``; ``chunk`` > 0: keys of its own chunk of that many tokens, counted from
+    the document's start; key tiles outside are not visited. ``gate`` (fp32 [T, hq]) multiplies every head's output.
+    Returns [T, hq * hd], in ``out`` (rows of any pitch) if given."""
+    if k.stride(0) != v.stride(0):
+        raise ValueError("flash_fwd_heads: k and v rows must have the same pitch")
+    t = q.shape[0]
+    if out is None:
+        out = torch.empty((t, hq * hd), dtype=q.dtype, device=q.device)
+    lse = torch.empty((hq, t), dtype=torch.float32, device=q.device)
+    call("icb_flash_fwd", ptr(q), ptr(k), ptr(v), ptr(out), ptr(lse), cu_seqlens.numel() - 1, int(max_seqlen), t, hq, hkv,
+         hd, q.stride(0), k.stride(0), ptr(cu_seqlens), 1, float(scale), dtype_code(q.dtype),
+         ptr(native.status_tensor(q.device)), stream_ptr(), 0.0, None, 0, int(window), ptr(gate), int(chunk), out.stride(0))
+    return out
 
 
 def flash_fwd_window(q: torch.Tensor, kv: torch.Tensor, heads: int, hd: int, cu_seqlens: torch.Tensor, max_seqlen: int,
                      *, scale: float, window: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Causal attention of separate projections ``q`` [T, heads * hd] and ``kv`` [T, 2 * heads * hd] (keys, then
-    values) within the documents of ``cu_seqlens`` (int32 [n + 1], the longest being ``max_seqlen``). ``window`` > 0:
-    query i sees keys j with ``i - j < window``; key tiles outside are not visited. ``gate`` (fp32 [T, heads])
-    multiplies every head's output. Returns [T, heads * hd]."""
-    t = q.shape[0]
-    es = kv.element_size()
-    out = torch.empty((t, heads * hd), dtype=q.dtype, device=q.device)
-    lse = torch.empty((heads, t), dtype=torch.float32, device=q.device)
-    call("icb_flash_fwd", ptr(q), kv.data_ptr(), kv.data_ptr() + heads * hd * es, ptr(out), ptr(lse),
-         cu_seqlens.numel() - 1, int(max_seqlen), t, heads, heads, hd, q.stride(0), kv.stride(0), ptr(cu_seqlens), 1,
-         float(scale), dtype_code(q.dtype), ptr(native.status_tensor(q.device)), stream_ptr(), 0.0, None, 0,
-         int(window), ptr(gate))
-    return out
+    """:func:`flash_fwd_heads` of separate projections ``q`` [T, heads * hd] and ``kv`` [T, 2 * heads * hd] (keys, then
+    values)."""
+    n = heads * hd
+    return flash_fwd_heads(q, kv[:, :n], kv[:, n:], heads, heads, hd, cu_seqlens, max_seqlen, scale=scale, window=window,
+                           gate=gate)
 
 
 def flash_bwd(dout: torch.Tensor, qkv: torch.Tensor, out: torch.Tensor, lse: torch.Tensor, hq: int, hkv: int, hd: int,

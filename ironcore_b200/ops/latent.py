@@ -21,20 +21,26 @@ native.register("icb_latent_attend", [P, P, P, P, P, P, P, I, I, I, I, I, I, F, 
 MMA_MAX_RANK = 512     # widest latent row of the tensor-core attention kernel
 
 
-def project(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """x [T, K] @ weight [N, K]^T (checkpoint orientation) -> [T, N] in ``out_dtype`` (default: x's)."""
+def project(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
+            bias: Optional[torch.Tensor] = None, transposed: bool = False) -> torch.Tensor:
+    """x [T, K] @ weight [N, K]^T (checkpoint orientation; ``transposed``: weight [K, N]) + bias -> [T, N] in
+    ``out_dtype`` (default: x's)."""
     out_dtype = out_dtype or x.dtype
     if use_native(x):
-        return kernels.mm_nt(x, weight, out_dtype=out_dtype)
+        return (kernels.mm_nn if transposed else kernels.mm_nt)(x, weight, out_dtype=out_dtype, bias=bias)
+    w = weight if transposed else weight.t()
     if x.dtype == torch.float32:
-        if not (x.is_cuda and torch.backends.cuda.matmul.allow_tf32):
-            return x @ weight.t()
-        torch.backends.cuda.matmul.allow_tf32 = False      # a 32-bit model is 32-bit, whatever training switched on
+        tf32 = x.is_cuda and torch.backends.cuda.matmul.allow_tf32
+        if tf32:
+            torch.backends.cuda.matmul.allow_tf32 = False      # a 32-bit model is 32-bit, whatever training switched on
         try:
-            return x @ weight.t()
+            y = x @ w
         finally:
-            torch.backends.cuda.matmul.allow_tf32 = True
-    return (x.float() @ weight.float().t()).to(out_dtype)
+            if tf32:
+                torch.backends.cuda.matmul.allow_tf32 = True
+        return y if bias is None else y + bias
+    y = x.float() @ w.float()
+    return (y if bias is None else y + bias.float()).to(out_dtype)
 
 
 def latent_norm(z: torch.Tensor, q_weight: torch.Tensor, c_weight: torch.Tensor, heads: int, eps: float, *,

@@ -15,7 +15,7 @@ from . import native
 from .native import call, dtype_code, ptr, stream_ptr
 
 P, I, L, F = native.P, native.I, native.L, native.F
-native.register("icb_stream_boundary", [P, P, L, L, F, P, P, P, L, P, L, P, P, P, P, P, P, I, F, P, P, L, P, P, P, P, P,
+native.register("icb_stream_boundary", [P, P, L, L, F, P, P, P, P, L, P, L, P, P, P, P, P, P, I, F, P, P, L, P, P, P, P, P,
                                         I, I, I, I, I, P])
 
 
@@ -44,6 +44,15 @@ class TokenEmbed:
 
 
 @dataclass
+class StreamAdd:
+    """What every stream gets on top where a pass of a looped block starts: ``vector`` fp32 [D] and, if given, the rows
+    of ``embed``."""
+
+    vector: torch.Tensor
+    embed: Optional[TokenEmbed] = None
+
+
+@dataclass
 class TokenShift:
     """Blend of a row with the previous token's: ``weight`` [D]; ``prev`` / ``state`` fp32 [slots, D] are the last
     value of every sequence before / after this batch (one tensor may serve as both if no sequence has more than one
@@ -58,29 +67,34 @@ class TokenShift:
 
 def boundary(source, read: torch.Tensor, norm_weight: torch.Tensor, groups: int, eps: float, *, width: int,
              dtype: torch.dtype, shift: Optional[TokenShift] = None, rows: Optional[torch.Tensor] = None,
-             keep_streams: bool = True) -> Tuple[Optional[torch.Tensor], torch.Tensor, Optional[torch.Tensor]]:
+             keep_streams: bool = True, add: Optional[StreamAdd] = None) -> Tuple[Optional[torch.Tensor], torch.Tensor, Optional[torch.Tensor]]:
     """``source`` is a :class:`StreamWrite` or a :class:`TokenEmbed`. Returns (streams, h, shifted h): the streams
-    after the write (None without ``keep_streams``), ``h`` [T, width] = grouped RMS norm of ``sum_s read[s] x_s`` and,
+    after the write and ``add`` (None without ``keep_streams``), ``h`` [T, width] = grouped RMS norm of ``sum_s read[s] x_s`` and,
     with ``shift``, its token-shifted form. ``rows`` (int32) selects rows of the source. ``width`` >= D pads with
     zeros."""
     first = isinstance(source, TokenEmbed)
     device = source.tokens.device if first else source.streams.device
     if device.type != "cuda":
-        return _boundary_reference(source, read, norm_weight, groups, eps, width, dtype, shift, rows, keep_streams)
+        return _boundary_reference(source, read, norm_weight, groups, eps, width, dtype, shift, rows, keep_streams, add)
     d = norm_weight.numel()
     s = source.streams if first else source.streams.shape[1]
     total = rows.numel() if rows is not None else (source.tokens.numel() if first else source.streams.shape[0])
     h = torch.empty((total, width), dtype=dtype, device=device)
     hs = torch.empty_like(h) if shift is not None else None
     x_out = torch.empty((total, s, d), dtype=torch.float32, device=device) if keep_streams else None
-    table = source.table if first else None
+    embed = source if first else (add.embed if add is not None else None)
+    if first and add is not None and add.embed is not None:
+        raise ValueError("stream boundary: the embedding is where the streams start, it cannot be added there too")
+    table = embed.table if embed is not None else None
     y = None if first else source.y
     gate = None if first else source.gate
     for t in (table, y, gate):
         if t is not None and (t.dtype != dtype or t.stride(-1) != 1):
             raise ValueError("stream boundary: table, y and gate share the activation dtype and have contiguous rows")
-    call("icb_stream_boundary", ptr(source.tokens) if first else None, ptr(table), table.stride(0) if first else 0,
-         table.shape[0] if first else 0, float(source.scale) if first else 0.0, None if first else ptr(source.streams), ptr(x_out), ptr(y),
+    call("icb_stream_boundary", ptr(embed.tokens) if embed is not None else None, ptr(table),
+         table.stride(0) if table is not None else 0, table.shape[0] if table is not None else 0,
+         float(embed.scale) if embed is not None else 0.0, ptr(add.vector) if add is not None else None,
+         None if first else ptr(source.streams), ptr(x_out), ptr(y),
          0 if first else y.stride(0), ptr(gate), gate.stride(0) if gate is not None else 0,
          None if gate is None else ptr(source.gate_bias), None if first else ptr(source.mix),
          None if first else ptr(source.out), ptr(rows), ptr(read), ptr(norm_weight), int(groups), float(eps), ptr(h),
@@ -96,7 +110,7 @@ def grouped_rms_norm_reference(x: torch.Tensor, weight: torch.Tensor, groups: in
     return parts.flatten(-2) * weight
 
 
-def _boundary_reference(source, read, norm_weight, groups, eps, width, dtype, shift, rows, keep_streams):
+def _boundary_reference(source, read, norm_weight, groups, eps, width, dtype, shift, rows, keep_streams, add):
     d = norm_weight.numel()
     if isinstance(source, TokenEmbed):
         x = (source.table[source.tokens, :d].float() * source.scale).unsqueeze(1).expand(-1, source.streams, -1)
@@ -105,6 +119,10 @@ def _boundary_reference(source, read, norm_weight, groups, eps, width, dtype, sh
         if source.gate is not None:
             y = y * torch.sigmoid(source.gate[:, :d].float() + source.gate_bias)
         x = torch.einsum("st,nsd->ntd", source.mix, source.streams) + source.out[:, None] * y[:, None]
+    if add is not None:
+        if add.embed is not None:
+            x = x + (add.embed.table[add.embed.tokens, :d].float() * add.embed.scale).unsqueeze(1)
+        x = x + add.vector
     if rows is not None:
         x = x[rows.long()]
     h = grouped_rms_norm_reference(torch.einsum("s,nsd->nd", read, x), norm_weight, groups, eps)

@@ -2,8 +2,8 @@
 pairs (``rl.dpo``: imported on demand, it pulls in the trainer)."""
 
 from .grpo import VocabSubsetReward, group_advantages, grpo_loss
-from .kv_cache import BlockKVCache, LatentCache
+from .kv_cache import BlockKVCache, LayerCache
 from .rollout import RolloutEngine
 from .sampling import sample_tokens
 
-__all__ = ["BlockKVCache", "LatentCache", "RolloutEngine", "VocabSubsetReward", "group_advantages", "grpo_loss", "sample_tokens"]
+__all__ = ["BlockKVCache", "LayerCache", "RolloutEngine", "VocabSubsetReward", "group_advantages", "grpo_loss", "sample_tokens"]

@@ -5,11 +5,11 @@ physical block of a sequence's i-th page and ``seq_lens[seq]`` its current lengt
 updated in place, so a captured CUDA graph of the decode step keeps reading the current state.
 
 * :class:`BlockKVCache` — keys and values, pools ``[num_blocks, block_size, kv_heads, head_dim]`` per layer.
-* :class:`LatentCache` — one latent row per token and layer run, plus a fixed-size state per sequence and layer run."""
+* :class:`LayerCache` — whatever the mixer of a layer run declares: rows per token, fixed-size states per sequence."""
 
 from __future__ import annotations
 
-from typing import Iterable, List, Optional, Sequence, Tuple
+from typing import Dict, Iterable, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -114,9 +114,8 @@ class PagedCache:
         blk = self.block_table[seq_ids.long(), page].long()
         return blk * self.block_size + (positions % self.block_size).long()
 
-    @property
-    def window(self) -> int:
-        """The furthest any layer looks back, the token itself included; 0 = to the first token."""
+    def visible_from(self, position: int) -> int:
+        """First token that any layer reads for a token at ``position``."""
         return 0
 
 
@@ -133,25 +132,32 @@ class BlockKVCache(PagedCache):
         return 2 * self.num_layers * self.kv_heads * self.head_dim * torch.empty((), dtype=self.dtype).element_size()
 
 
-class LatentCache(PagedCache):
-    """``latent[run]``: rows [num_blocks * block_size, row width of that run]. ``shift_state[run]``: fp32
-    [max_seqs, state width], the last normed input of every sequence. With a ``window``, pages that no layer can see
-    any more go back to the free list while a sequence is still running."""
+class LayerCache(PagedCache):
+    """``rows[run][name]``: [num_blocks * block_size, width]; ``states[run][name]``: [max_seqs, ...], one per sequence, as
+    the run's :class:`~ironcore_b200.layers.mixer.CacheSpec` in ``specs`` declares them. Pages that no layer reads any more
+    go back to the free list while a sequence is still running. A state belongs to whoever holds the sequence number;
+    mixers take it for zeros at position 0."""
 
-    def __init__(self, row_widths: Sequence[int], state_width: int, *, max_seqs: int, max_seq_len: int,
-                 block_size: int = 16, num_blocks: Optional[int] = None, window: int = 0, dtype=torch.bfloat16,
-                 device="cuda"):
+    def __init__(self, specs: Sequence, *, max_seqs: int, max_seq_len: int, block_size: int = 16,
+                 num_blocks: Optional[int] = None, dtype=torch.bfloat16, device="cuda"):
         if num_blocks is None:
             num_blocks = max_seqs * ((max_seq_len + block_size - 1) // block_size)
         super().__init__(num_blocks, block_size, max_seqs, max_seq_len, device)
-        self._window, self.dtype, self.row_widths = int(window), dtype, list(row_widths)
-        self.latent = [torch.zeros((num_blocks * block_size, w), dtype=dtype, device=self.device) for w in row_widths]
-        self.shift_state = [torch.zeros((max_seqs, state_width), dtype=torch.float32, device=self.device)
-                            for _ in row_widths]
+        self.specs, self.dtype = list(specs), dtype
+        self.rows: List[Dict[str, torch.Tensor]] = [
+            {name: torch.zeros((num_blocks * block_size, w), dtype=dtype, device=self.device) for name, w in s.rows.items()}
+            for s in self.specs]
+        self.states: List[Dict[str, torch.Tensor]] = [
+            {name: torch.zeros((max_seqs, *shape), dtype=dt or dtype, device=self.device)
+             for name, (shape, dt) in s.states.items()} for s in self.specs]
 
-    @property
-    def window(self) -> int:
-        return self._window
+    def visible_from(self, position: int) -> int:
+        reach = [lo for lo in (s.visible_from(position) for s in self.specs) if lo is not None]
+        return min(reach) if reach else position
 
     def bytes_per_token(self) -> int:
-        return sum(self.row_widths) * torch.empty((), dtype=self.dtype).element_size()
+        return sum(sum(s.rows.values()) for s in self.specs) * torch.empty((), dtype=self.dtype).element_size()
+
+    def bytes_per_sequence(self) -> int:
+        """Fixed-size states of one sequence."""
+        return sum(t[0].numel() * t.element_size() for run in self.states for t in run.values())

@@ -156,8 +156,8 @@ class TransformerProgram:
 
 
 class StreamProgram:
-    """Residual-stream models: latent rows and shift states in a :class:`LatentCache`, fp32 logits. Pages hold 64 tokens
-    unless asked otherwise: a latent row is narrow, and the decode kernel copies a page with one box per 64 columns."""
+    """Residual-stream models: a :class:`LayerCache` of whatever the mixers keep, fp32 logits. Pages hold 64 tokens unless
+    asked otherwise: a latent row is narrow, and its decode kernel copies a page with one box per 64 columns."""
 
     PAGE = 64
 

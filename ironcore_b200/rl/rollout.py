@@ -101,9 +101,8 @@ class RolloutEngine:
     # ------------------------------------------------------------------ batches
     def _make_room(self, seqs: List[int], counts: List[int]):
         cache = self.cache
-        if cache.window > 0:
-            for s in seqs:
-                cache.drop_before(s, max(0, cache.length(s) - cache.window + 1))
+        for s in seqs:
+            cache.drop_before(s, cache.visible_from(cache.length(s)))
         cache.reserve_many((s, cache.length(s) + n) for s, n in zip(seqs, counts))
 
     def _rows(self, seqs: List[int], counts: List[int], tokens: torch.Tensor, want: Optional[List[int]]) -> torch.Tensor:
