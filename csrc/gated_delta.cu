@@ -129,7 +129,11 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const DeltaPrepArgs<
       float f[4];
       load_f32<4>(at, f);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) f[i] = expf(rate * softplus_f32(f[i] + bias[i]));
+      for (int i = 0; i < 4; ++i) {
+        const float x = rate * softplus_f32(f[i] + bias[i]);
+        // factors near one act thousands of times: in fp32 models they are rounded once
+        f[i] = sizeof(T) == 4 ? (float)exp((double)x) : expf(x);
+      }
       store_f32<4>(at, f);
     }
     return;

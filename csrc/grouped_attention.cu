@@ -1,7 +1,7 @@
 // Attention with grouped key / value heads over a paged cache, the parts around the tensor-core kernels:
 //
 //  * rope_cache  : one pass over the packed projection of a batch: rotates the heads of q and k in place (partial rotary,
-//                  pairs (i, i + dims / 2), angles in fp32), writes the rotated keys and the values to their cache rows
+//                  pairs (i, i + dims / 2)), writes the rotated keys and the values to their cache rows
 //                  and turns the gate logits into factors.
 //  * attend_rows : one query row of one head per CTA against its visible cache rows, any head sizes, bf16 or fp32, all
 //                  arithmetic in fp32. It serves fp32 models and shapes that the tensor-core kernels do not take.
@@ -19,7 +19,7 @@ struct RopeCacheArgs {
   T* v_cache;               // [slots, G x VD]
   const long long* slots;   // cache row of a token, negative: none
   const int* pos;
-  const float* freq;        // [half]
+  const double* freq;       // [half] radians per position
   float* gate;              // [rows, H] or null
   float gate_scale;
   int H, G, KD, VD, half;   // half: rotated pairs per head
@@ -32,10 +32,14 @@ __global__ void __launch_bounds__(kRopeThreads) rope_cache_kernel(const RopeCach
   extern __shared__ float cs[];   // [half] cos, [half] sin
   const int r = blockIdx.x;
   T* z = a.z + (size_t)r * a.ldz;
-  const float p = (float)a.pos[r];
+  const double p = (double)a.pos[r];
   for (int i = threadIdx.x; i < a.half; i += kRopeThreads) {
+    // an fp32 product loses position * 2^-24 radians, which grows along a sequence: product and reduction to one turn in
+    // fp64, once per row and pair
+    double turn = p * a.freq[i] * 0.15915494309189535;
+    turn -= rint(turn);
     float s, c;
-    sincosf(p * a.freq[i], &s, &c);
+    sincosf((float)(turn * 6.283185307179586), &s, &c);
     cs[i] = c;
     cs[a.half + i] = s;
   }
@@ -198,10 +202,10 @@ __global__ void __launch_bounds__(kAttendThreads) attend_rows_kernel(const Atten
 using namespace icb;
 
 // z [rows, ldz] (bf16 or fp32): [q: H x KD | k: G x KD | v: G x VD | H gate logits]. The first 2 * half elements of every
-// q and k head rotate in place by pos * freq (pairs i, i + half); keys and values go to rows `slots` (int64, negative:
+// q and k head rotate in place by pos * freq (fp64 [half]; pairs i, i + half); keys and values go to rows `slots` (int64, negative:
 // skip) of the caches; gate (fp32 [rows, H], optional) = gate_scale * sigmoid(logit). KD, VD, ldz: multiples of 8.
 ICB_API int icb_rope_cache(void* z, long long ldz, void* k_cache, void* v_cache, const long long* slots, const int* pos,
-                           const float* freq, int half, float* gate, float gate_scale, int rows, int H, int G, int KD,
+                           const double* freq, int half, float* gate, float gate_scale, int rows, int H, int G, int KD,
                            int VD, int dtype, void* stream) {
   if (rows <= 0) return 0;
   if (G < 1 || H % G || KD % 8 || VD % 8 || ldz % 8 || half < 0 || 2 * half > KD || half > 4096) return -2;

@@ -6,7 +6,9 @@
 // and C rows arrive by asynchronous copies while the tile before is computed. What depends on one element only
 // (softplus, dt u on the way in; D u, silu and the conversion on the way out) is done once per element by all threads;
 // the loop over time in between touches shared memory and registers alone. A channel's states are spread over
-// `lanes` neighbouring lanes with NS each; exp runs in the base-2 domain with log2(e) folded into A.
+// `lanes` neighbouring lanes with NS each. In 16-bit models exp runs in the base-2 domain with log2(e) folded into A; in
+// fp32 models a state that hardly decays would add up that function's error over thousands of tokens, so there
+// S <- S + (expm1(dt A) S + dt u B).
 // Decoding is the same kernel with one row per sequence and wider channel blocks.
 #include "host_common.h"
 #include "rows.cuh"
@@ -41,6 +43,12 @@ __device__ __forceinline__ float exp2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+template <typename T>
+__device__ __forceinline__ float scan_step(float x, float s, float in) {
+  if constexpr (sizeof(T) == 4) return s + fmaf(expm1f(x), s, in);
+  return fmaf(exp2_approx(x), s, in);
 }
 
 // Shared memory of one tile buffer, in bytes; CH channels, NB = lanes * NS padded states.
@@ -113,7 +121,7 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Scan
         const float l[4] = {al.x, al.y, al.z, al.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e)
-          if (n0 + i + e < a.N) a2[i + e] = -expf(l[e]) * 1.4426950408889634f;
+          if (n0 + i + e < a.N) a2[i + e] = sizeof(T) == 4 ? -expf(l[e]) : -expf(l[e]) * 1.4426950408889634f;
         if (!seq.fresh) {
           const float4 u = *reinterpret_cast<const float4*>(st + i);
           s[i] = u.x; s[i + 1] = u.y; s[i + 2] = u.z; s[i + 3] = u.w;
@@ -155,10 +163,10 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(const Scan
       for (int i = 0; i < NS; i += 4) {
         const float4 b = *reinterpret_cast<const float4*>(pb + i);
         const float4 k = *reinterpret_cast<const float4*>(pc + i);
-        s[i] = fmaf(exp2_approx(dt * a2[i]), s[i], du * b.x);
-        s[i + 1] = fmaf(exp2_approx(dt * a2[i + 1]), s[i + 1], du * b.y);
-        s[i + 2] = fmaf(exp2_approx(dt * a2[i + 2]), s[i + 2], du * b.z);
-        s[i + 3] = fmaf(exp2_approx(dt * a2[i + 3]), s[i + 3], du * b.w);
+        s[i] = scan_step<T>(dt * a2[i], s[i], du * b.x);
+        s[i + 1] = scan_step<T>(dt * a2[i + 1], s[i + 1], du * b.y);
+        s[i + 2] = scan_step<T>(dt * a2[i + 2], s[i + 2], du * b.z);
+        s[i + 3] = scan_step<T>(dt * a2[i + 3], s[i + 3], du * b.w);
         y0 = fmaf(s[i], k.x, y0);
         y1 = fmaf(s[i + 1], k.y, y1);
         y0 = fmaf(s[i + 2], k.z, y0);

@@ -19,9 +19,9 @@ native.register("icb_attend_rows", [P, L, P, P, P, I, I, P, P, P, P, L, I, I, I,
 
 
 def rotary_frequencies(dims: int, base: float) -> torch.Tensor:
-    """fp32 [dims / 2]: base^(-2 i / dims), rounded once."""
+    """Radians per position of every rotated pair, fp64 [dims / 2]: base^(-2 i / dims)."""
     i = torch.arange(dims // 2, dtype=torch.float64)
-    return (float(base) ** (-2.0 * i / dims)).float()
+    return float(base) ** (-2.0 * i / dims)
 
 
 def first_visible(position: torch.Tensor, window: int, chunk: int) -> torch.Tensor:
@@ -46,8 +46,8 @@ def rope_cache(z: torch.Tensor, freq: torch.Tensor, positions: torch.Tensor, *, 
         call("icb_rope_cache", ptr(z), z.stride(0), ptr(k_cache), ptr(v_cache), ptr(slots), ptr(positions), ptr(freq), half,
              ptr(gate), float(gate_scale or 0.0), t, heads, groups, kd, vd, dtype_code(z.dtype), stream_ptr())
         return gate
-    angle = positions.float()[:, None] * freq
-    c, s = torch.cos(angle)[:, None], torch.sin(angle)[:, None]
+    angle = positions.double()[:, None] * freq
+    c, s = torch.cos(angle).float()[:, None], torch.sin(angle).float()[:, None]
     qk = z[:, :(heads + groups) * kd].view(t, heads + groups, kd)
     u, v = qk[..., :half].float(), qk[..., half:2 * half].float()
     qk[..., :half], qk[..., half:2 * half] = (u * c - v * s).to(z.dtype), (v * c + u * s).to(z.dtype)
