@@ -311,8 +311,9 @@ def main(argv=None):
     ap.add_argument("--norm-gather", dest="norm_gather", default="auto", choices=["auto", "on", "off"],
                     help="fuse reduce-scatter + RMSNorm + all-gather across the norm boundaries (auto: TP >= 4)")
     ap.add_argument("--workload", default="train", choices=["train", "serving"],
-                    help="train: the headline step; serving: prefill and decode of the residual-stream family beside "
+                    help="train: the headline step; serving: prefill and decode of a residual-stream family beside "
                          "the transformer of equal size (see benchmarks/serving.py)")
+    ap.add_argument("--family", default="tetepel", choices=["tetepel", "kedavik"], help="serving: which family")
     ap.add_argument("--size", default=None, choices=["2k", "4k"], help="serving: one size instead of all")
     ap.add_argument("--kernels-only", dest="kernels_only", action="store_true", help="serving: kernels only")
     args = ap.parse_args(argv)
