@@ -26,15 +26,13 @@ SIZES = {
 }
 
 
-# Kedavik beside the transformer of the same width: selective-scan layers (inner = 2 width) without feed-forward alternate
-# with attention + delta rule layers, so it has more and smaller layers at about the same number of weights
+# Kedavik beside the transformer of the same width, heads and depth: selective-scan layers (inner = 2 width) without
+# feed-forward alternate with layers of attention (a quarter of the key / value heads) beside the delta rule
 KEDAVIK_SIZES = {
-    "4k": dict(width=4096, heads=16, kv=4, head=128, chunk=2048, d_heads=16, d_head=128, inner=8192, state=16, dt_rank=256,
-               conv=4, rank=128, ff=11008, vocab=32000, layers=6, prompt=4096, seqs=4, decode_seqs=64, decode_prompt=2000,
-               llama=dict(heads=32, layers=4)),
-    "2k": dict(width=2048, heads=8, kv=2, head=128, chunk=1024, d_heads=8, d_head=128, inner=4096, state=16, dt_rank=128,
-               conv=4, rank=128, ff=5632, vocab=32000, layers=12, prompt=4096, seqs=8, decode_seqs=128, decode_prompt=1000,
-               llama=dict(heads=16, layers=8)),
+    "4k": dict(width=4096, heads=32, kv=8, head=128, chunk=2048, d_heads=32, d_head=128, inner=8192, state=16, dt_rank=256,
+               conv=4, rank=128, ff=11008, vocab=32000, layers=4, prompt=4096, seqs=4, decode_seqs=64, decode_prompt=2000),
+    "2k": dict(width=2048, heads=16, kv=4, head=128, chunk=1024, d_heads=16, d_head=128, inner=4096, state=16, dt_rank=128,
+               conv=4, rank=128, ff=5632, vocab=32000, layers=8, prompt=4096, seqs=8, decode_seqs=128, decode_prompt=1000),
 }
 
 
@@ -104,7 +102,7 @@ def bench_models(family: str, size: str, steps: int, warmup: int, report) -> Non
 
     z = (SIZES if family == "tetepel" else KEDAVIK_SIZES)[size]
     for label, build in ((family, _stream_model if family == "tetepel" else _kedavik_model), ("llama", _llama_model)):
-        model, cfg = build({**z, **z.get("llama", {})} if label == "llama" else z)
+        model, cfg = build(z)
         params = sum(p.numel() for p in model.parameters())
         gen = torch.Generator().manual_seed(3)
         native.reset_launches()
@@ -188,7 +186,7 @@ def bench_kedavik_kernels(size: str, report) -> None:
     dev, bf, f32, rand, emit = "cuda", torch.bfloat16, dict(dtype=torch.float32), _rand, _emitter(size, report)
     d, ff, taps, n, inner = (z[k] for k in ("width", "ff", "conv", "state", "inner"))
     h, g, hd, e, k = (z[x] for x in ("heads", "kv", "head", "d_heads", "d_head"))
-    lh = z["llama"]["heads"]
+    lh = h
     for t in (z["seqs"] * z["prompt"], z["decode_seqs"]):
         few = t == z["decode_seqs"]
         n_seq = t if few else z["seqs"]

@@ -11,14 +11,17 @@ template <typename T>
 constexpr int kVec = 16 / (int)sizeof(T);
 
 template <typename T>
-__device__ __forceinline__ void load_row(const T* p, float (&f)[kVec<T>]) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
+__device__ __forceinline__ void unpack_row(const uint4 u, float (&f)[kVec<T>]) {
   if constexpr (sizeof(T) == 4) {
     f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
   } else {
     const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y), c = unpack_bf16x2(u.z), d = unpack_bf16x2(u.w);
     f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
   }
+}
+template <typename T>
+__device__ __forceinline__ void load_row(const T* p, float (&f)[kVec<T>]) {
+  unpack_row<T>(*reinterpret_cast<const uint4*>(p), f);
 }
 template <typename T>
 __device__ __forceinline__ void store_row(T* p, const float (&f)[kVec<T>]) {
@@ -45,7 +48,50 @@ __device__ __forceinline__ void store_f32(float* p, const float (&f)[V]) {
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// An activation of a 16-bit tensor: fast exp and division. Of an fp32 tensor: full precision.
+template <typename T>
+__device__ __forceinline__ float silu_of(float x) {
+  if constexpr (sizeof(T) == 4) return silu_f32(x);
+  return __fdividef(x, 1.f + __expf(-x));
+}
+// log(1 + exp(x)). The 16-bit models' form sums log(1 + e) = 2 artanh(e / (2 + e)) for e = exp(-|x|) <= 1 as a series
+// (argument at most 1/3, first term left out below 1.5e-7 of the sum).
+template <typename T>
+__device__ __forceinline__ float softplus_of(float x) {
+  if constexpr (sizeof(T) == 4) return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+  const float e = __expf(-fabsf(x)), s = __fdividef(e, 2.f + e), q = s * s;
+  float p = fmaf(q, 1.f / 11.f, 1.f / 9.f);
+  p = fmaf(q, p, 1.f / 7.f);
+  p = fmaf(q, p, 1.f / 5.f);
+  p = fmaf(q, p, 1.f / 3.f);
+  p = fmaf(q, p, 1.f);
+  return fmaxf(x, 0.f) + 2.f * s * p;
+}
+
+// Two fp32 values in a register pair: one instruction multiplies and adds both.
+struct Pair {
+  unsigned long long v;
+};
+__device__ __forceinline__ Pair pair_of(float lo, float hi) {
+  Pair p;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(p.v) : "f"(lo), "f"(hi));
+  return p;
+}
+__device__ __forceinline__ float2 pair_values(Pair p) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(p.v));
+  return f;
+}
+__device__ __forceinline__ Pair pair_mul(Pair a, Pair b) {
+  Pair d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d.v) : "l"(a.v), "l"(b.v));
+  return d;
+}
+__device__ __forceinline__ Pair pair_fma(Pair a, Pair b, Pair c) {
+  Pair d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return d;
+}
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(gmem) : "memory");
@@ -113,46 +159,73 @@ __device__ __forceinline__ void conv_input(const ConvArgs<T>& a, int r, int befo
   }
 }
 
-// Convolution and silu of kVec<T> channels of row r. TAPS > 0 fixes the number of taps and takes the weights of `w`
-// from registers (load_conv_weights); 0 reads both at run time.
-template <typename T, int TAPS>
-struct ConvWeights {
-  float w[TAPS > 0 ? TAPS : 1][kVec<T>];
-};
-template <typename T, int TAPS>
-__device__ __forceinline__ void load_conv_weights(const ConvArgs<T>& a, int ch, ConvWeights<T, TAPS>& k) {
-  if constexpr (TAPS > 0) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load_f32<kVec<T>>(a.w + (size_t)(TAPS - 1 - j) * a.C + ch, k.w[j]);
-  }
+// The same values as they are stored: one 16-byte piece.
+template <typename T>
+__device__ __forceinline__ uint4 conv_piece(const ConvArgs<T>& a, int r, int before, int slot, int pos, int j, int ch) {
+  if (j <= before) return *reinterpret_cast<const uint4*>(a.x + (size_t)(r - j) * a.ldx + ch);
+  if (pos - j >= 0)
+    return *reinterpret_cast<const uint4*>(a.state + ((size_t)slot * (a.taps - 1) + (a.taps - 1 - (j - before))) * a.C + ch);
+  return make_uint4(0u, 0u, 0u, 0u);
 }
+
+// Convolution and silu of kVec<T> neighbouring channels along consecutive rows. TAPS > 0: the weights and the last
+// TAPS - 1 inputs stay in registers, a row costs one load. TAPS == 0: any number of taps, everything read per row.
 template <typename T, int TAPS>
-__device__ __forceinline__ void conv_silu_row(const ConvArgs<T>& a, const ConvWeights<T, TAPS>& k, int r, int before,
-                                              int slot, int pos, int ch, float (&out)[kVec<T>]) {
-  constexpr int V = kVec<T>;
-  if (a.bias != nullptr) load_f32<V>(a.bias + ch, out);
-  else {
-#pragma unroll
-    for (int v = 0; v < V; ++v) out[v] = 0.f;
-  }
-  const int taps = TAPS > 0 ? TAPS : a.taps;
-#pragma unroll
-  for (int j = 0; j < taps; ++j) {
-    float x[V];
-    conv_input<T>(a, r, before, slot, pos, j, ch, x);
+struct ConvLane {
+  static constexpr int V = kVec<T>;
+  static constexpr int H = TAPS > 1 ? TAPS - 1 : 1;
+  float w[TAPS > 0 ? TAPS : 1][V];      // [j]: of the input j tokens back
+  uint4 past[H];                        // [j]: the input j + 1 tokens back
+  int ch;
+
+  __device__ __forceinline__ void init(const ConvArgs<T>& a, int channel) {
+    ch = channel;
     if constexpr (TAPS > 0) {
 #pragma unroll
-      for (int v = 0; v < V; ++v) out[v] = fmaf(k.w[j][v], x[v], out[v]);
-    } else {
-      float w[V];
-      load_f32<V>(a.w + (size_t)(taps - 1 - j) * a.C + ch, w);
-#pragma unroll
-      for (int v = 0; v < V; ++v) out[v] = fmaf(w[v], x[v], out[v]);
+      for (int j = 0; j < TAPS; ++j) load_f32<V>(a.w + (size_t)(TAPS - 1 - j) * a.C + ch, w[j]);
     }
   }
+  // before row r, when the row before it was not the last one this lane has seen of the same sequence
+  __device__ __forceinline__ void refill(const ConvArgs<T>& a, int r, int before, int slot, int pos) {
+    if constexpr (TAPS > 1) {
 #pragma unroll
-  for (int v = 0; v < V; ++v) out[v] = silu_f32(out[v]);
-}
+      for (int j = 1; j < TAPS; ++j) past[j - 1] = conv_piece<T>(a, r, before, slot, pos, j, ch);
+    }
+  }
+  __device__ __forceinline__ uint4 fetch(const ConvArgs<T>& a, int r) const {
+    return *reinterpret_cast<const uint4*>(a.x + (size_t)r * a.ldx + ch);
+  }
+  __device__ __forceinline__ void row(const ConvArgs<T>& a, uint4 x, int r, int before, int slot, int pos, float (&out)[V]) {
+    if (a.bias != nullptr) load_f32<V>(a.bias + ch, out);
+    else {
+#pragma unroll
+      for (int v = 0; v < V; ++v) out[v] = 0.f;
+    }
+    float f[V];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int j = TAPS - 1; j > 0; --j) {
+        unpack_row<T>(past[j - 1], f);
+#pragma unroll
+        for (int v = 0; v < V; ++v) out[v] = fmaf(w[j][v], f[v], out[v]);
+        if (j > 1) past[j - 1] = past[j - 2];
+      }
+      unpack_row<T>(x, f);
+#pragma unroll
+      for (int v = 0; v < V; ++v) out[v] = fmaf(w[0][v], f[v], out[v]);
+      if constexpr (TAPS > 1) past[0] = x;
+    } else {
+      for (int j = 0; j < a.taps; ++j) {
+        conv_input<T>(a, r, before, slot, pos, j, ch, f);
+        load_f32<V>(a.w + (size_t)(a.taps - 1 - j) * a.C + ch, w[0]);
+#pragma unroll
+        for (int v = 0; v < V; ++v) out[v] = fmaf(w[0][v], f[v], out[v]);
+      }
+    }
+#pragma unroll
+    for (int v = 0; v < V; ++v) out[v] = silu_of<T>(out[v]);
+  }
+};
 
 // The inputs that a sequence's next token needs, from its last row r of this batch. Entry e takes what is newer than
 // itself only, so one thread may do this in place in ascending order.
@@ -165,12 +238,12 @@ __device__ __forceinline__ void conv_keep(const ConvArgs<T>& a, int r, int befor
   }
 }
 
-// How many consecutive rows a thread takes: long runs keep the taps in L1, but the machine should be full first.
-inline int conv_run(long long rows, long long threads_per_row, int sms) {
-  const long long fill = (long long)sms * 2048;
-  long long run = rows * threads_per_row / fill;
+// How many consecutive rows a thread takes: long runs share the weights and the first inputs, but the machine
+// (`resident` threads per SM) should be full two times over first.
+inline int conv_run(long long rows, long long threads_per_row, int sms, int resident) {
+  long long run = rows * threads_per_row / (2LL * sms * resident);
   if (run < 1) run = 1;
-  if (run > 32) run = 32;
+  if (run > 64) run = 64;
   return (int)run;
 }
 

@@ -5,32 +5,50 @@
 
 namespace icb {
 
+constexpr int kConvAhead = 4;      // rows whose loads are in flight per thread
+
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) short_conv_kernel(const ConvArgs<T> a, T* __restrict__ y, long long ldy, int rows,
                                                          int run, int keep) {
   constexpr int V = kVec<T>;
   const int per_row = a.C / V;
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  const int r0 = (int)(idx / per_row) * run;
-  if (r0 >= rows) return;
-  const int ch = (int)(idx % per_row) * V;
+  const long long at = idx / per_row * run;
+  if (at >= rows) return;
+  const int r0 = (int)at, r1 = min(rows, r0 + run);
   const int most = (TAPS > 0 ? TAPS : a.taps) - 1;
-  ConvWeights<T, TAPS> k;
-  load_conv_weights<T, TAPS>(a, ch, k);
-  int before = rows_before(a.seqs, r0, most);
-  const int r1 = min(rows, r0 + run);
-  int slot = a.seqs[r0];
-  for (int r = r0; r < r1; ++r) {
-    if (r > r0) {
-      const int s = a.seqs[r];
-      before = s == slot ? min(before + 1, most) : 0;
-      slot = s;
+  ConvLane<T, TAPS> lane;
+  lane.init(a, (int)(idx % per_row) * V);
+  int before = rows_before(a.seqs, r0, most), slot = a.seqs[r0];
+  lane.refill(a, r0, before, slot, a.pos[r0]);
+  for (int g = r0; g < r1; g += kConvAhead) {
+    uint4 x[kConvAhead];
+    int s[kConvAhead];
+#pragma unroll
+    for (int i = 0; i < kConvAhead; ++i)
+      if (g + i < r1) {
+        x[i] = lane.fetch(a, g + i);
+        s[i] = a.seqs[g + i];
+      }
+#pragma unroll
+    for (int i = 0; i < kConvAhead; ++i) {
+      const int r = g + i;
+      if (r >= r1) break;
+      if (r > r0) {
+        if (s[i] == slot) {
+          before = min(before + 1, most);
+        } else {
+          before = 0;
+          slot = s[i];
+          lane.refill(a, r, 0, slot, a.pos[r]);
+        }
+      }
+      const int pos = TAPS > 0 && !keep ? 0 : a.pos[r];      // the register window does not ask
+      float out[V];
+      lane.row(a, x[i], r, before, slot, pos, out);
+      store_row<T>(y + (size_t)r * ldy + lane.ch, out);
+      if (keep) conv_keep<T>(a, r, before, slot, pos, lane.ch);
     }
-    const int pos = a.pos[r];
-    float out[V];
-    conv_silu_row<T, TAPS>(a, k, r, before, slot, pos, ch, out);
-    store_row<T>(y + (size_t)r * ldy + ch, out);
-    if (keep) conv_keep<T>(a, r, before, slot, pos, ch);
   }
 }
 
@@ -49,11 +67,13 @@ template <typename T>
 static int launch_conv(const ConvArgs<T>& a, T* y, long long ldy, const int* cu, int n, int rows, cudaStream_t st) {
   const int per_row = a.C / kVec<T>;
   if (y != nullptr) {
-    const int run = cu == nullptr ? 1 : conv_run(rows, per_row, num_sms());
+    const int run = cu == nullptr ? 1 : conv_run(rows, per_row, num_sms(), 2 * 256);
     const long long threads = (long long)((rows + run - 1) / run) * per_row;
     const int blocks = (int)((threads + 255) / 256);
     const int keep = cu == nullptr && a.taps > 1;     // every row is its sequence's only one: nobody else reads the state
     if (a.taps == 4) short_conv_kernel<T, 4><<<blocks, 256, 0, st>>>(a, y, ldy, rows, run, keep);
+    else if (a.taps == 3) short_conv_kernel<T, 3><<<blocks, 256, 0, st>>>(a, y, ldy, rows, run, keep);
+    else if (a.taps == 2) short_conv_kernel<T, 2><<<blocks, 256, 0, st>>>(a, y, ldy, rows, run, keep);
     else short_conv_kernel<T, 0><<<blocks, 256, 0, st>>>(a, y, ldy, rows, run, keep);
     int rc = check_launch("short_conv_kernel");
     if (rc) return rc;
