@@ -24,7 +24,7 @@ class SelectiveScanSpec:
     def __post_init__(self):
         if min(self.inner, self.state, self.dt_rank, self.conv) < 1:
             raise ValueError(f"selective scan: sizes must be positive ({self})")
-        OR.scan_lanes(self.state, 1)
+        OR.scan_lanes(self.state)      # refuses what the kernel cannot hold
 
 
 class SelectiveScan(Branch):

@@ -93,10 +93,10 @@ def _conv_reference(x, weight, bias, state, rows, keep):
 
 
 # --------------------------------------------------------------------------- selective scan
-def scan_lanes(n: int, rows_per_sequence: int) -> int:
-    """States per lane of the scan kernel (a channel's states are spread over a power of two of lanes, sixteen at most).
-    Long runs of rows want as few idle lanes as possible and many states per lane, since every lane also pays for the
-    per-channel work; one row at a time is bound by the state's bytes."""
+def scan_lanes(n: int) -> int:
+    """States per lane of the scan kernel (a channel's states are spread over a power of two of lanes, sixteen at most):
+    few idle lanes, several states per lane, since every lane also pays for the per-channel work, but not so many that the
+    machine runs out of warps (measured: 8 of 16)."""
     best, cost = 0, float("inf")
     for ns in (8, 4, 12, 16, 32):
         lanes = 1
@@ -104,7 +104,7 @@ def scan_lanes(n: int, rows_per_sequence: int) -> int:
             lanes *= 2
         if lanes > 16:
             continue
-        c = lanes * (ns + (3.0 if rows_per_sequence > 1 else 1.0)) + (8.0 if ns > 16 else 0.0)
+        c = lanes * (ns + 3.0) + (16.0 if ns > 16 else 8.0 if ns > 8 else 0.0)
         if c < cost:
             best, cost = ns, c
     if best == 0:
@@ -123,7 +123,7 @@ def selective_scan(u: torch.Tensor, dt: torch.Tensor, z: torch.Tensor, bc: torch
         call("icb_selective_scan", ptr(u), u.stride(0), ptr(dt), dt.stride(0), ptr(z), z.stride(0), ptr(bc), bc.stride(0),
              int(b_col), int(c_col), ptr(dt_bias), ptr(a_log), ptr(d), ptr(state), ptr(out), out.stride(0),
              ptr(rows.seqs), ptr(rows.positions), ptr(rows.cu), rows.count, rows.longest, c, int(n),
-             per_lane or scan_lanes(n, rows.longest), dtype_code(u.dtype), stream_ptr())
+             per_lane or scan_lanes(n), dtype_code(u.dtype), stream_ptr())
         return
     a = -torch.exp(a_log[:, :n])
     step = TF.softplus(dt + dt_bias, threshold=1e9)
