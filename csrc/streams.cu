@@ -82,8 +82,9 @@ __device__ __forceinline__ void store_vec(T* p, const float (&f)[V]) {
   }
 }
 
-// S_ > 0 fixes the number of streams at compile time; 0 reads it from the arguments.
-template <typename T, int S_, int V>
+// S_ > 0 fixes the number of streams at compile time; 0 reads it from the arguments. EXTRA: embedding rows or a vector come
+// in (always so at the first boundary).
+template <typename T, int S_, int V, bool EXTRA>
 __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(const StreamArgs a) {
   extern __shared__ __align__(16) float row_smem[];     // u [D], then (with a shift) the previous row's h [D]
   __shared__ float s_mix[kMaxStreams * kMaxStreams], s_out[kMaxStreams], s_in[kMaxStreams];
@@ -93,7 +94,7 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
   const int D = a.D, G = a.groups, gs = D / G;
   float* su = row_smem;
   float* sprev = row_smem + D;
-  const bool write_step = a.x_in != nullptr;
+  const bool write_step = !EXTRA || a.x_in != nullptr;
   for (int i = threadIdx.x; i < S * S; i += blockDim.x) s_mix[i] = write_step ? a.mix[i] : 0.f;
   for (int i = threadIdx.x; i < S; i += blockDim.x) {
     s_out[i] = write_step ? a.out[i] : 0.f;
@@ -123,7 +124,7 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
       if (first && a.row_pos[r] > 0) before = a.prev + (size_t)seq * D;
     }
     const T* table_row = nullptr;
-    if (a.table != nullptr) {
+    if (EXTRA && a.table != nullptr) {
       const long long id = a.tokens[src];
       if (id >= 0 && id < a.table_rows) table_row = reinterpret_cast<const T*>(a.table) + id * a.ld_table;
     }
@@ -142,12 +143,12 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
         float e[V];                                     // what every stream gets besides the write step
 #pragma unroll
         for (int v = 0; v < V; ++v) e[v] = 0.f;
-        if (table_row != nullptr) {
+        if (EXTRA && table_row != nullptr) {
           load_vec<T, V>(table_row + col, e);
 #pragma unroll
           for (int v = 0; v < V; ++v) e[v] *= a.table_scale;
         }
-        if (a.add != nullptr) {
+        if (EXTRA && a.add != nullptr) {
           float p[V];
           load_vec<float, V>(a.add + col, p);
 #pragma unroll
@@ -239,9 +240,9 @@ __global__ void __launch_bounds__(kStreamMaxWarps * 32) stream_boundary_kernel(c
   }
 }
 
-template <typename T, int S_, int V>
+template <typename T, int S_, int V, bool EXTRA>
 static int launch_stream_v(const StreamArgs& a, int blocks, int threads, size_t smem, cudaStream_t st) {
-  auto kern = stream_boundary_kernel<T, S_, V>;
+  auto kern = stream_boundary_kernel<T, S_, V, EXTRA>;
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return -(int)e;
@@ -251,8 +252,12 @@ static int launch_stream_v(const StreamArgs& a, int blocks, int threads, size_t 
 }
 template <typename T, int S_>
 static int launch_stream_s(const StreamArgs& a, bool wide, int blocks, int threads, size_t smem, cudaStream_t st) {
-  return wide ? launch_stream_v<T, S_, 4>(a, blocks, threads, smem, st)
-              : launch_stream_v<T, S_, 1>(a, blocks, threads, smem, st);
+  const bool extra = a.table != nullptr || a.add != nullptr;
+  if (wide)
+    return extra ? launch_stream_v<T, S_, 4, true>(a, blocks, threads, smem, st)
+                 : launch_stream_v<T, S_, 4, false>(a, blocks, threads, smem, st);
+  return extra ? launch_stream_v<T, S_, 1, true>(a, blocks, threads, smem, st)
+               : launch_stream_v<T, S_, 1, false>(a, blocks, threads, smem, st);
 }
 template <typename T>
 static int launch_stream(const StreamArgs& a, bool wide, int blocks, int threads, size_t smem, cudaStream_t st) {
