@@ -107,7 +107,7 @@ def test_gated_delta_kernels(dtype, heads, groups, dim, vdim, taps):
 
     conv, sizes = 2 * groups * dim + heads * vdim, dict(groups=groups, heads=heads, dim=dim, vdim=vdim)
     valid = vdim - 3
-    for spans, decode in ((MIXTURE, False), (ONE_EACH, True)):
+    for spans, decode in ((MIXTURE, False), (_spans(3), False), (ONE_EACH, True)):      # few rows, and enough for two launches
         t = sum(c for _, _, c in spans)
         x, beta = _rand(t, conv + 8, dtype=dtype), _rand(t, heads, seed=1, dtype=dtype)
         cw, a = _rand(taps, conv, seed=2), _rand(t, heads * dim, seed=3)
